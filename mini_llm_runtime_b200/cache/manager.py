@@ -2,7 +2,7 @@
 of fixed-size state per request.
 
 What the model's mixers need is declared per cache entry (one entry per run step that writes):
-``KVCacheNeed`` (all earlier keys, or a window of them) or ``StateNeed`` (a fixed-size tensor per
+``KVCacheNeed`` (all earlier keys, a window of them, or the position's own chunk) or ``StateNeed`` (a fixed-size tensor per
 request).  Entries with the same key/value geometry and window form a *group*; each group has
 its own page pool, its own allocator and, per request, its own block table, because a windowed
 group gives pages back while the request still runs and a full group does not.
@@ -78,7 +78,7 @@ class CacheGroup:
     def kept_pages(self) -> int:
         """Leading pages of a windowed group that are never given back while the request lives:
         those that hold the positions the window always keeps visible."""
-        return _ceil_div(self.need.keep_first, self.page_size) if self.need.window is not None else 0
+        return _ceil_div(self.need.keep_first, self.page_size) if self.need.span is not None else 0
 
 
 @dataclass
@@ -204,9 +204,10 @@ class CacheManager:
     def pages_for_lifetime(self, group: CacheGroup, lifetime_tokens: int) -> int:
         """Most pages of ``group`` a request of ``lifetime_tokens`` cached tokens holds at once."""
         full = _ceil_div(lifetime_tokens, self.page_size)
-        if group.window is None:
+        span = group.need.span
+        if span is None:
             return full
-        live = _ceil_div(group.window - 1 + self.max_step_tokens, self.page_size) + 1 + group.kept_pages
+        live = _ceil_div(span - 1 + self.max_step_tokens, self.page_size) + 1 + group.kept_pages
         return min(full, live)
 
     def lifetime_pages(self, lifetime_tokens: int) -> tuple[int, ...]:
@@ -355,11 +356,10 @@ class CacheManager:
             request.pending = None
             for group in self.groups:
                 request.step_new_pages[group.index] = []
-                if group.window is None:
+                if group.need.span is None:
                     continue
-                # The next query sits at position `committed` and sees keys > committed - window.
-                lowest_needed = request.committed - group.window + 1
-                first_needed_page = max(0, lowest_needed) // self.page_size
+                # The next query sits at position `committed`: keys outside its window or chunk are seen no more.
+                first_needed_page = group.need.lowest_visible(request.committed) // self.page_size
                 pages = request.pages[group.index]
                 gone = []
                 # the pages of the positions a window keeps visible for good are never given back

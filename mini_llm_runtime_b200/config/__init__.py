@@ -5,11 +5,12 @@ from .registry import (Architecture, architecture_of, config_from_dict, known_ar
                        load_config, register_architecture, unregister_architecture)
 from .rozesun import RozesunConfig, RozesunLayer, rozesun_model_spec
 from .spec import LayerSpec, ModelSpec, PartSpec, RunStep
+from .vetevik import VetevikConfig, VetevikLayer, vetevik_model_spec
 from .zazasun import ZazasunConfig, ZazasunLayer, zazasun_model_spec
 
 __all__ = [
     "Architecture", "BopilornConfig", "BopilornLayer", "LayerSpec", "ModelSpec", "PartSpec", "Qwen2Config", "RatilornConfig", "RatilornLayer", "RozesunConfig", "RozesunLayer",
-    "RunStep", "ZazasunConfig", "ZazasunLayer",
+    "RunStep", "VetevikConfig", "VetevikLayer", "ZazasunConfig", "ZazasunLayer",
     "architecture_of", "bopilorn_model_spec", "config_from_dict", "known_architectures", "load_config",
-    "qwen2_model_spec", "ratilorn_model_spec", "register_architecture", "rozesun_model_spec", "unregister_architecture", "zazasun_model_spec",
+    "qwen2_model_spec", "ratilorn_model_spec", "register_architecture", "rozesun_model_spec", "unregister_architecture", "vetevik_model_spec", "zazasun_model_spec",
 ]

@@ -18,6 +18,7 @@ from .qwen2 import Qwen2Config, qwen2_model_spec
 from .ratilorn import RatilornConfig, ratilorn_model_spec
 from .rozesun import RozesunConfig, rozesun_model_spec
 from .spec import ModelSpec
+from .vetevik import VetevikConfig, vetevik_model_spec
 from .zazasun import ZazasunConfig, zazasun_model_spec
 
 
@@ -87,3 +88,4 @@ register_architecture(ZazasunConfig.architecture, ZazasunConfig.from_dict, zazas
 register_architecture(RozesunConfig.architecture, RozesunConfig.from_dict, rozesun_model_spec)
 register_architecture(BopilornConfig.architecture, BopilornConfig.from_dict, bopilorn_model_spec)
 register_architecture(RatilornConfig.architecture, RatilornConfig.from_dict, ratilorn_model_spec)
+register_architecture(VetevikConfig.architecture, VetevikConfig.from_dict, vetevik_model_spec)

@@ -50,6 +50,7 @@ class RunStep:
     cache: int
     writes_cache: bool = True
     offset_row: int | None = None     # row of the model's offset table added to the stream before the layer
+    add_embedding: bool = False       # the embedding's rows are added to the stream again before the layer
 
 
 @dataclass(frozen=True)
@@ -77,6 +78,8 @@ class ModelSpec:
                 raise ValueError(f"run step {position} has a negative cache entry")
             if step.offset_row is not None and self.offsets is None:
                 raise ValueError(f"run step {position} asks for an offset, but the model has no offset table")
+            if step.offset_row is not None and step.add_embedding:
+                raise ValueError(f"run step {position} asks for an offset and for the embedding's rows")
             if step.writes_cache:
                 if step.cache in writers:
                     raise ValueError(f"cache entry {step.cache} is written by run steps "

@@ -344,11 +344,49 @@ static int row_threads(int width) {
   return 64;
 }
 
+// Rows of `heads` heads of `dim` entries (a column range of wider rows) into the pages of a cache:
+// pool[page][head][offset] = x[row][head], slot = page * page_size + offset.  A thread per piece of `piece` bytes.
+template <typename PIECE>
+__global__ void __launch_bounds__(256)
+store_heads_kernel(const uint8_t* x, long long row_bytes, const long long* slots, uint8_t* pool, long long total, int heads,
+                   int pieces_per_head, int page_size) {
+  pdl_trigger();
+  pdl_wait();
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= total) return;
+  const int per_row = heads * pieces_per_head;
+  const long long row = idx / per_row;
+  const int within = (int)(idx - row * per_row), head = within / pieces_per_head, c = within - head * pieces_per_head;
+  const long long slot = slots[row];
+  if (slot < 0) return;
+  const long long page = slot / page_size, offset = slot - page * page_size;
+  const PIECE value = __ldcg(reinterpret_cast<const PIECE*>(x + row * row_bytes) + within);
+  reinterpret_cast<PIECE*>(pool)[((page * heads + head) * page_size + offset) * pieces_per_head + c] = value;
+}
+
 }  // namespace mlr
 
 using namespace mlr;
 
 MLR_DEFINE_PDL_SWITCH
+
+// x: rows of heads * dim entries of `itemsize` (2 or 4) bytes spaced row_stride entries apart; slots: int64
+// [rows]; pool: [pages, heads, page_size, dim].
+MLR_EXPORT int mlr_store_heads(const void* x, long long row_stride, const long long* slots, void* pool, int rows, int heads,
+                               int dim, int page_size, int itemsize, cudaStream_t stream) {
+  if (rows == 0) return MLR_OK;
+  if (rows < 0 || heads <= 0 || dim <= 0 || page_size <= 0 || (itemsize != 2 && itemsize != 4)) return MLR_BAD_SIZE;
+  const long long row_bytes = row_stride * itemsize;
+  const int head_bytes = dim * itemsize;
+  const bool wide = head_bytes % 16 == 0 && row_bytes % 16 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)pool & 15) == 0;
+  const int pieces = wide ? head_bytes / 16 : dim;
+  const long long total = (long long)rows * heads * pieces, blocks = (total + 255) / 256;
+  if (blocks > 0x7fffffffLL) return MLR_TOO_LARGE;
+  auto kernel = wide ? store_heads_kernel<uint4> : itemsize == 4 ? store_heads_kernel<unsigned int> : store_heads_kernel<unsigned short>;
+  launch_kernel(kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (const uint8_t*)x, row_bytes, slots, (uint8_t*)pool,
+                total, heads, pieces, page_size);
+  return launch_status();
+}
 
 MLR_EXPORT int mlr_embedding(const int* ids, const void* table, void* out, int rows, int width,
                              int vocab, int dtype, cudaStream_t stream) {

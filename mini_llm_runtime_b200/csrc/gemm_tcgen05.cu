@@ -139,6 +139,7 @@ struct GemmParams {
   // the stacked matrix [groups * N, K]; rows at or beyond the end row are computed and not written;
   // an entry whose group is negative is unused.  The list is device memory written by an earlier kernel.
   const int* group_tiles;
+  const float* row_scale;    // grouped form: factor of every row's product (before the gate), or null
 };
 
 constexpr int MAX_STAGES = 8;
@@ -501,6 +502,14 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           tmem_issue_load16(from + 64 + c0 + 16, u + 16);
           tmem_wait_loads();
           if (m >= row_limit) continue;
+          if (grouped && p.row_scale != nullptr) {
+            const float scale = __ldcg(p.row_scale + m);
+#pragma unroll
+            for (int c = 0; c < 32; ++c) {
+              g[c] = __float_as_uint(scale * __uint_as_float(g[c]));
+              u[c] = __float_as_uint(scale * __uint_as_float(u[c]));
+            }
+          }
 #pragma unroll
           for (int q = 0; q < 32; q += 16) {
             const int n0 = (tile_y * (BN / 128) + block) * 64 + c0 + q;
@@ -543,6 +552,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         }
         const int m = a_row0 + accumulator * TILE_ROWS + row;
         if (m >= row_limit) continue;
+        if (grouped && p.row_scale != nullptr) {
+          const float scale = __ldcg(p.row_scale + m);
+#pragma unroll
+          for (int c = 0; c < ROUND; ++c) v[c] *= scale;
+        }
 #pragma unroll
         for (int q = 0; q < ROUND; q += 16) {
           const int n0 = n_tile0 + c00 + q;
@@ -847,6 +861,7 @@ MLR_EXPORT int mlr_gemm_tcgen05(const void* x, const void* w, const void* bias, 
   p.counters = counters;
   p.error_word = error_word;
   p.group_tiles = nullptr;
+  p.row_scale = nullptr;
   if (plan.splits > 1 && (scratch == nullptr || counters == nullptr)) return MLR_BAD_SIZE;
   if (swiglu) {
     if (M <= 16) return launch<16, true, true>(x, w, p, plan.splits, stream);
@@ -893,11 +908,12 @@ static int launch_grouped(const void* x, const void* w, const GemmParams& p, int
 // or 256 where N is a multiple of 256: two accumulators from one load of the weight tile, one CTA
 // per SM) rows of one group, group < 0 for unused entries; it may be written by the kernel just
 // before this one.  A 128-row load may run into the next group's rows (or past the last row: zeros);
-// those rows are computed and dropped.  N % BN need not hold only without swiglu: a weight tile that would run into
+// those rows are computed and dropped.  `row_scale` (float32 [rows] or null) multiplies each row's product,
+// before the gate (the same as scaling the rows of x).  N % BN need not hold only without swiglu: a weight tile that would run into
 // the next group's rows is loaded but its columns beyond N are never written.
 MLR_EXPORT int mlr_gemm_tcgen05_grouped(const void* x, const void* w, void* out, const int* tiles, int max_tiles, int rows,
                                         int groups, int N, int K, int out_f32, int swiglu, int tile_rows,
-                                        int* error_word, cudaStream_t stream) {
+                                        const float* row_scale, int* error_word, cudaStream_t stream) {
   if (rows == 0 || max_tiles == 0) return MLR_OK;
   if (rows < 0 || max_tiles < 0 || groups <= 0 || N <= 0 || K <= 0 || tiles == nullptr) return MLR_BAD_SIZE;
   if (K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return MLR_BAD_ALIGNMENT;
@@ -928,6 +944,7 @@ MLR_EXPORT int mlr_gemm_tcgen05_grouped(const void* x, const void* w, void* out,
   p.counters = nullptr;
   p.error_word = error_word;
   p.group_tiles = tiles;
+  p.row_scale = row_scale;
   if (tall) return swiglu ? launch_grouped<256, true, 2 * TILE_ROWS>(x, w, p, rows, groups, max_tiles, stream)
                           : launch_grouped<256, false, 2 * TILE_ROWS>(x, w, p, rows, groups, max_tiles, stream);
   if (swiglu) return wide ? launch_grouped<256, true>(x, w, p, rows, groups, max_tiles, stream)

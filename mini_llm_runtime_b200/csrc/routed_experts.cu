@@ -7,7 +7,8 @@
 //                        largest choice scores (1: its largest), only experts of the `keep` best groups can be chosen; the `top` largest
 //                        choice scores win (ties: the lower index); the weights are the winners' s,
 //                        divided by their sum + renorm_eps if asked.  chosen int32 [rows, top], weights float32.
-// mlr_expert_hidden      for every (row, chosen expert) pair p: hidden[p] = act(Wg_e x) * (Wu_e x), a warp
+// mlr_expert_hidden      for every (row, chosen expert) pair p: hidden[p] = act(Wg_e x) * (Wu_e x), x times the
+//                        pair's weight where weights belong to the experts' inputs; a warp
 //                        per four outputs, the dot products split over the lanes in a fixed order.
 // mlr_expert_down        out[row] = sum_t weights[row, t] * (Wd_e(t) hidden[row * top + t]) in float32, t
 //                        ascending: a warp per four output columns, the chosen experts one after the other.
@@ -299,8 +300,8 @@ constexpr int DOWN_PER_CTA = EXPERT_WARPS * PER_WARP;
 // of the same outputs (block == ff: all gate rows first).
 template <typename T>
 __global__ void __launch_bounds__(EXPERT_WARPS * 32)
-expert_hidden_kernel(const T* x, const int* chosen, const T* __restrict__ gate_up, T* hidden, int K, int ff, int top,
-                     int block, int act, int wide) {
+expert_hidden_kernel(const T* x, const int* chosen, const float* weights, const T* __restrict__ gate_up, T* hidden, int K,
+                     int ff, int top, int block, int act, int wide) {
   pdl_trigger();
   extern __shared__ __align__(16) float xs[];      // [K]
   const int pair = blockIdx.x;
@@ -308,6 +309,7 @@ expert_hidden_kernel(const T* x, const int* chosen, const T* __restrict__ gate_u
   pdl_wait();
   const int row = pair / top;
   const int expert = chosen[pair];
+  const float scale = weights != nullptr ? __ldcg(weights + pair) : 1.f;      // of the expert's input
   for (int k = threadIdx.x; k < K; k += blockDim.x) xs[k] = load_as_float(x + (size_t)row * K + k);
   __syncthreads();
   const T* w = gate_up + (size_t)expert * 2 * ff * K;
@@ -328,8 +330,8 @@ expert_hidden_kernel(const T* x, const int* chosen, const T* __restrict__ gate_u
 #pragma unroll
     for (int i = 0; i < PER_WARP; ++i)
       if (i == lane) {
-        gate = sums[i];
-        up = sums[PER_WARP + i];
+        gate = scale * sums[i];
+        up = scale * sums[PER_WARP + i];
       }
     float value;
     if (act == 1) {
@@ -369,7 +371,7 @@ expert_down_kernel(const T* hidden, const int* chosen, const float* weights, con
     for (int i = 0; i < PER_WARP; ++i) rows[i] = down + ((size_t)expert * N + min(n0 + i, N - 1)) * ff;
     float y[PER_WARP];
     warp_dots<PER_WARP, T>(rows, hs + (size_t)t * pitch, ff, lane, wide != 0, y);
-    const float weight = weights[(size_t)row * top + t];
+    const float weight = weights != nullptr ? weights[(size_t)row * top + t] : 1.f;
 #pragma unroll
     for (int i = 0; i < PER_WARP; ++i) total[i] = fmaf(weight, y[i], total[i]);
   }
@@ -388,8 +390,8 @@ expert_down_kernel(const T* hidden, const int* chosen, const float* weights, con
 // to max_tiles.  The order inside an expert's run is not fixed (atomics); every pair's result is
 // computed from its own row alone, so the order changes no number.
 __global__ void __launch_bounds__(1024)
-sort_pairs_kernel(const int* chosen, int* place, int* token_of, int* tiles, int pairs, int top, int experts, int tile_rows,
-                  int max_tiles) {
+sort_pairs_kernel(const int* chosen, const float* weights, int* place, int* token_of, float* sorted_weights, int* tiles,
+                  int pairs, int top, int experts, int tile_rows, int max_tiles) {
   pdl_trigger();
   extern __shared__ int counts[];        // [experts] counts, [experts + 1] starts, [experts] cursors
   int* starts = counts + experts;
@@ -423,6 +425,7 @@ sort_pairs_kernel(const int* chosen, int* place, int* token_of, int* tiles, int 
     const int at = atomicAdd(&cursor[chosen[p]], 1);
     place[p] = at;
     token_of[at] = p / top;
+    if (sorted_weights != nullptr) sorted_weights[at] = __ldcg(weights + p);
   }
 }
 
@@ -450,7 +453,7 @@ combine_pairs_kernel(const float* y, const int* place, const float* weights, flo
   for (int n = threadIdx.x; n < N; n += blockDim.x) {
     float total = 0.f;
     for (int t = 0; t < top; ++t)
-      total = fmaf(weights[(size_t)row * top + t], __ldcg(y + (size_t)place[(size_t)row * top + t] * N + n), total);
+      total = fmaf(weights != nullptr ? weights[(size_t)row * top + t] : 1.f, __ldcg(y + (size_t)place[(size_t)row * top + t] * N + n), total);
     out[(size_t)row * N + n] = total;
   }
 }
@@ -509,9 +512,10 @@ MLR_EXPORT int mlr_route_experts(const void* x, const float* router, const float
   return launch_status();
 }
 
-// x: [rows, K]; chosen: int32 [rows * top]; gate_up: [experts, 2 * ff, K]; hidden: [rows * top, ff]; all
-// floating tensors in `dtype`.  act: 0 silu, 1 the tanh form of gelu.
-MLR_EXPORT int mlr_expert_hidden(const void* x, const int* chosen, const void* gate_up, void* hidden, int rows, int K, int ff,
+// x: [rows, K]; chosen: int32 [rows * top]; weights: float32 [rows * top] that multiply the experts' inputs, or
+// null; gate_up: [experts, 2 * ff, K]; hidden: [rows * top, ff]; all other floating tensors in `dtype`.  act: 0
+// silu, 1 the tanh form of gelu.
+MLR_EXPORT int mlr_expert_hidden(const void* x, const int* chosen, const float* weights, const void* gate_up, void* hidden, int rows, int K, int ff,
                                  int top, int block, int act, int dtype, cudaStream_t stream) {
   if (rows == 0) return MLR_OK;
   if (rows < 0 || K <= 0 || ff <= 0 || top <= 0 || block <= 0 || ff % block != 0) return MLR_BAD_SIZE;
@@ -523,7 +527,7 @@ MLR_EXPORT int mlr_expert_hidden(const void* x, const int* chosen, const void* g
       cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
       if (err != cudaSuccess) return (int)err;
     }
-    launch_kernel(kernel, grid, threads, shared, stream, xt, chosen, wt, ht, K, ff, top, block, act, wide);
+    launch_kernel(kernel, grid, threads, shared, stream, xt, chosen, weights, wt, ht, K, ff, top, block, act, wide);
     return launch_status();
   };
   const bool aligned = ((uintptr_t)gate_up & 15) == 0;
@@ -534,7 +538,7 @@ MLR_EXPORT int mlr_expert_hidden(const void* x, const int* chosen, const void* g
   return MLR_BAD_DTYPE;
 }
 
-// hidden: [rows * top, ff]; down: [experts, N, ff] in `dtype`; weights: float32 [rows * top]; out: float32 [rows, N].
+// hidden: [rows * top, ff]; down: [experts, N, ff] in `dtype`; weights: float32 [rows * top] or null (ones); out: float32 [rows, N].
 MLR_EXPORT int mlr_expert_down(const void* hidden, const int* chosen, const float* weights, const void* down, float* out,
                                int rows, int N, int ff, int top, int dtype, cudaStream_t stream) {
   if (rows == 0) return MLR_OK;
@@ -556,14 +560,16 @@ MLR_EXPORT int mlr_expert_down(const void* hidden, const int* chosen, const floa
   return MLR_BAD_DTYPE;
 }
 
-// chosen: int32 [pairs]; place: int32 [pairs]; token_of: int32 [pairs]; tiles: int32 [max_tiles, 3].
-MLR_EXPORT int mlr_sort_pairs(const int* chosen, int* place, int* token_of, int* tiles, int pairs, int top, int experts,
+// chosen: int32 [pairs]; place: int32 [pairs]; token_of: int32 [pairs]; tiles: int32 [max_tiles, 3]; weights
+// (float32 [pairs]) and sorted_weights (the same in the order of places) may both be null.
+MLR_EXPORT int mlr_sort_pairs(const int* chosen, const float* weights, int* place, int* token_of, float* sorted_weights,
+                              int* tiles, int pairs, int top, int experts,
                               int tile_rows, int max_tiles, cudaStream_t stream) {
   if (pairs == 0) return MLR_OK;
   if (pairs < 0 || top <= 0 || experts <= 0 || tile_rows <= 0 || max_tiles <= 0) return MLR_BAD_SIZE;
   const size_t shared = sizeof(int) * (3 * (size_t)experts + 1);
   if (shared > 48 * 1024) return MLR_TOO_LARGE;
-  launch_kernel(sort_pairs_kernel, dim3(1), dim3(1024), shared, stream, chosen, place, token_of, tiles, pairs, top, experts,
+  launch_kernel(sort_pairs_kernel, dim3(1), dim3(1024), shared, stream, chosen, weights, place, token_of, sorted_weights, tiles, pairs, top, experts,
                 tile_rows, max_tiles);
   return launch_status();
 }

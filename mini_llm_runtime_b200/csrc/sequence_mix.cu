@@ -488,6 +488,25 @@ MLR_EXPORT int mlr_gated_recurrence(int mode, const float* r, long long r_stride
   return mode == 0 || mode == 1 ? MLR_BAD_DTYPE : MLR_BAD_SIZE;
 }
 
+// out = y / rms(y) * weight * silu(gate) head by head: y float32 [rows, heads * vdim]; gate: float32 rows of that
+// width spaced gate_stride apart, or null; weight: float32 [vdim], shared by the heads.
+MLR_EXPORT int mlr_gated_head_norm(const float* y, const float* gate, long long gate_stride, const float* weight, void* out,
+                                   int rows, int heads, int vdim, float eps, int out_dtype, cudaStream_t stream) {
+  if (rows == 0) return MLR_OK;
+  if (rows < 0 || heads <= 0 || vdim <= 0) return MLR_BAD_SIZE;
+  const long long items = (long long)rows * heads;
+  const dim3 grid((unsigned)((items + 3) / 4));
+  if (out_dtype == MLR_F32)
+    launch_kernel(recurrence_finish_kernel<float>, grid, dim3(128), 0, stream, y, gate, gate_stride, weight, 0, (float*)out,
+                  items, heads, vdim, eps);
+  else if (out_dtype == MLR_BF16)
+    launch_kernel(recurrence_finish_kernel<bf16>, grid, dim3(128), 0, stream, y, gate, gate_stride, weight, 0, (bf16*)out,
+                  items, heads, vdim, eps);
+  else
+    return MLR_BAD_DTYPE;
+  return launch_status();
+}
+
 MLR_EXPORT int mlr_add_residual(float* residual, const float* a, const float* b, long long count, cudaStream_t stream) {
   if (count == 0) return MLR_OK;
   if (count < 0) return MLR_BAD_SIZE;

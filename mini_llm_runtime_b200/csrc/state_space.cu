@@ -16,6 +16,7 @@
 // mlr_gated_group_norm   out = RMSnorm_parts(y * silu(z)) * weight: the row is cut into `parts` equal parts,
 //                        each divided by its own root mean square (eps inside the root).
 #include "common.cuh"
+#include "copy_async.cuh"
 
 #include <type_traits>
 
@@ -117,16 +118,6 @@ struct ScanArgs {
   const int *seg_q_start, *seg_q_len, *seg_slot;
   int heads, vdim, n, groups;
 };
-
-// Asynchronous copies into shared memory (the data never passes through registers, and the thread goes on).
-__device__ __forceinline__ void copy_async_4(float* dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_async_16(float* dst, const float* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // SL: threads that share one value channel's state (a power of two; SL * SCAN_NPT >= n).  Lane l of a warp
 // holds 16 entries of channel p = l / SL: the pieces of four entries number s, s + SL, s + 2 SL, s + 3 SL with
@@ -300,14 +291,14 @@ MLR_EXPORT int mlr_causal_conv(const float* u, long long u_stride, const float* 
                                float* out, const int* seg_q_start, const int* seg_q_len, const int* seg_slot, int segments,
                                int max_q_len, int channels, int taps, int act, cudaStream_t stream) {
   if (segments == 0) return MLR_OK;
-  if (segments < 0 || max_q_len <= 0 || channels <= 0 || taps < 2) return MLR_BAD_SIZE;
+  if (segments < 0 || max_q_len <= 0 || channels <= 0 || taps < 1) return MLR_BAD_SIZE;
   if (taps > MAX_TAPS || segments > 65535) return MLR_TOO_LARGE;
   const int chunks = (max_q_len + CONV_TOKENS - 1) / CONV_TOKENS;
   if (chunks > 65535) return MLR_TOO_LARGE;
   launch_kernel(causal_conv_kernel, dim3((channels + 127) / 128, segments, chunks), dim3(128), 0, stream, u, u_stride, weight,
                 bias, states, out, seg_q_start, seg_q_len, seg_slot, channels, taps, act);
   int status = launch_status();
-  if (status != MLR_OK || max_q_len == 1) return status;
+  if (status != MLR_OK || max_q_len == 1 || taps == 1) return status;      // one tap carries nothing
   launch_kernel(carry_kernel, dim3((channels + 127) / 128, segments), dim3(128), 0, stream, u, u_stride, states, seg_q_start,
                 seg_q_len, seg_slot, channels, taps);
   return launch_status();

@@ -13,7 +13,9 @@
 // mlr_rms_norm_step        the same pass for sublayers that are normalised on their way into the stream by
 //                          an RMS norm (no centering, no bias): x += delta / rms(delta) * dw, then
 //                          out = x / rms(x) * w, or the rows of x as they are in the compute dtype when
-//                          no w is given (the input of a sublayer that reads the stream itself).
+//                          no w is given (the input of a sublayer that reads the stream itself); an offset
+//                          (a vector, or rows) may be added in between, and rms may be taken over equal parts
+//                          of the row.
 // mlr_normed_mean          out = factor * (a / rms(a) * wa + b / rms(b) * wb) for two float32 inputs.
 // mlr_clamped_gate         y = g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit) and
 //                          u = clamp(up, -limit, limit), on rows of gate/up blocks.
@@ -307,24 +309,36 @@ __device__ __forceinline__ float row_inverse_rms(const float* values, int width,
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-rms_norm_step_kernel(float* x, const float* delta, const float* __restrict__ dw, const float* __restrict__ w,
-                     T* __restrict__ out, int width, float eps) {
+rms_norm_step_kernel(float* x, const float* delta, const float* __restrict__ dw, const float* offset, int offset_rows,
+                     const float* __restrict__ w, T* __restrict__ out, int width, int groups, float eps) {
   pdl_trigger();
   extern __shared__ float staged[];      // [width] + 32
   float* scratch = staged + width;
   const size_t base = (size_t)blockIdx.x * width;
+  const int first = groups > 1 ? (int)(blockIdx.x % groups) * width : 0;      // of this part, in the whole row
+  if (dw != nullptr) dw += first;
+  if (w != nullptr) w += first;
+  if (offset != nullptr) offset += offset_rows ? base : (size_t)first;
   pdl_wait();
   if (delta != nullptr) {
     for (int d = threadIdx.x; d < width; d += blockDim.x) staged[d] = __ldcg(delta + base + d);
     __syncthreads();
     const float rstd = row_inverse_rms(staged, width, eps, scratch);
     for (int d = threadIdx.x; d < width; d += blockDim.x) {
-      const float v = __ldcg(x + base + d) + staged[d] * rstd * dw[d];
+      float v = __ldcg(x + base + d) + staged[d] * rstd * dw[d];
+      if (offset != nullptr) v += __ldcg(offset + d);
       staged[d] = v;
       x[base + d] = v;
     }
   } else {
-    for (int d = threadIdx.x; d < width; d += blockDim.x) staged[d] = __ldcg(x + base + d);
+    for (int d = threadIdx.x; d < width; d += blockDim.x) {
+      float v = __ldcg(x + base + d);
+      if (offset != nullptr) {
+        v += __ldcg(offset + d);
+        x[base + d] = v;
+      }
+      staged[d] = v;
+    }
   }
   if (out == nullptr) return;
   if (w == nullptr) {
@@ -360,15 +374,19 @@ normed_mean_kernel(const float* a, const float* __restrict__ wa, const float* b,
 // pieces per thread, every operand asked for before the first is used (one trip to memory).
 template <typename T, int THREADS>
 __global__ void __launch_bounds__(THREADS)
-rms_norm_step_row_kernel(float* x, const float* delta, const float* __restrict__ dw, const float* __restrict__ w,
-                         T* __restrict__ out, int width, float eps) {
+rms_norm_step_row_kernel(float* x, const float* delta, const float* __restrict__ dw, const float* offset, int offset_rows,
+                         const float* __restrict__ w, T* __restrict__ out, int width, int groups, float eps) {
   pdl_trigger();
   __shared__ float scratch[THREADS / 32];
   constexpr int CH = 4;
   const int pieces = width >> 2;
   const size_t base = (size_t)blockIdx.x * width;
+  const int first = groups > 1 ? (int)(blockIdx.x % groups) * width : 0;      // of this part, in the whole row
+  if (dw != nullptr) dw += first;
+  if (w != nullptr) w += first;
+  if (offset != nullptr) offset += offset_rows ? base : (size_t)first;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 dwv[CH], wv[CH], dv[CH], xv[CH];
+  float4 dwv[CH], wv[CH], dv[CH], xv[CH], ov[CH];
 #pragma unroll
   for (int j = 0; j < CH; ++j) {
     const int c = threadIdx.x + THREADS * j;
@@ -383,6 +401,7 @@ rms_norm_step_row_kernel(float* x, const float* delta, const float* __restrict__
     const bool in = c < pieces;
     dv[j] = in && delta != nullptr ? __ldcg(reinterpret_cast<const float4*>(delta + base) + c) : zero;
     xv[j] = in ? __ldcg(reinterpret_cast<const float4*>(x + base) + c) : zero;
+    ov[j] = in && offset != nullptr ? __ldcg(reinterpret_cast<const float4*>(offset) + c) : zero;
   }
   if (delta != nullptr) {
     float sq = 0.f;
@@ -393,6 +412,12 @@ rms_norm_step_row_kernel(float* x, const float* delta, const float* __restrict__
     for (int j = 0; j < CH; ++j) {
       xv[j].x += dv[j].x * rstd * dwv[j].x; xv[j].y += dv[j].y * rstd * dwv[j].y;
       xv[j].z += dv[j].z * rstd * dwv[j].z; xv[j].w += dv[j].w * rstd * dwv[j].w;
+    }
+  }
+  if (delta != nullptr || offset != nullptr) {
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+      xv[j].x += ov[j].x; xv[j].y += ov[j].y; xv[j].z += ov[j].z; xv[j].w += ov[j].w;
       if (threadIdx.x + THREADS * j < pieces) store4(x + base + 4 * (threadIdx.x + THREADS * j), xv[j]);
     }
   }
@@ -565,34 +590,40 @@ MLR_EXPORT int mlr_layer_norm_step(float* x, const float* delta, const float* dw
   return MLR_BAD_DTYPE;
 }
 
-// x: float32 [rows, width], updated in place when delta is given.  delta: float32 [rows, width] or null
-// (then dw is not read); dw, w: float32 [width]; out: [rows, width] in out_dtype or null.  With out and no
-// w, out receives the rows of x (after the add) as they are.
-MLR_EXPORT int mlr_rms_norm_step(float* x, const float* delta, const float* dw, const float* w, void* out, int rows,
-                                 int width, float eps, int out_dtype, cudaStream_t stream) {
+// x: float32 [rows, width], updated in place when delta or offset is given.  delta: float32 [rows, width] or
+// null (then dw is not read); dw, w: float32 [width]; offset: float32 [rows, width] (offset_rows != 0) or
+// [width], or null; out: [rows, width] in out_dtype or null.  With out and no w, out receives the rows of x
+// (after the adds) as they are.  Each row is cut into `groups` equal parts that are divided by their own root
+// mean squares.
+MLR_EXPORT int mlr_rms_norm_step(float* x, const float* delta, const float* dw, const float* offset, int offset_rows,
+                                 const float* w, void* out, int rows, int width, int groups, float eps, int out_dtype,
+                                 cudaStream_t stream) {
   if (rows == 0) return MLR_OK;
-  if (rows < 0 || width <= 0 || (delta != nullptr && dw == nullptr)) return MLR_BAD_SIZE;
+  if (rows < 0 || width <= 0 || groups <= 0 || width % groups != 0 || (delta != nullptr && dw == nullptr)) return MLR_BAD_SIZE;
+  if ((long long)rows * groups > 0x7fffffffll) return MLR_TOO_LARGE;
+  rows *= groups;      // from here on a part is a row of its own
+  width /= groups;
   const size_t shared = sizeof(float) * ((size_t)width + 32);
   if (shared > 200 * 1024) return MLR_TOO_LARGE;
   auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  const bool few = rows <= 64 && width % 4 == 0 && width <= 8192 && aligned(x) && aligned(delta) && aligned(dw) && aligned(w) &&
-                   aligned(out);
+  const bool few = rows <= 64 * groups && width % 4 == 0 && width <= 8192 && aligned(x) && aligned(delta) && aligned(dw) &&
+                   aligned(offset) && aligned(w) && aligned(out);
   auto launch = [&](auto kernel, auto* typed_out) -> int {
     using T = std::remove_pointer_t<decltype(typed_out)>;
     if (few) {
       if (width <= 2048)
-        launch_kernel(rms_norm_step_row_kernel<T, 128>, dim3(rows), dim3(128), 0, stream, x, delta, dw, w, typed_out, width, eps);
+        launch_kernel(rms_norm_step_row_kernel<T, 128>, dim3(rows), dim3(128), 0, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);
       else if (width <= 4096)
-        launch_kernel(rms_norm_step_row_kernel<T, 256>, dim3(rows), dim3(256), 0, stream, x, delta, dw, w, typed_out, width, eps);
+        launch_kernel(rms_norm_step_row_kernel<T, 256>, dim3(rows), dim3(256), 0, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);
       else
-        launch_kernel(rms_norm_step_row_kernel<T, 512>, dim3(rows), dim3(512), 0, stream, x, delta, dw, w, typed_out, width, eps);
+        launch_kernel(rms_norm_step_row_kernel<T, 512>, dim3(rows), dim3(512), 0, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);
       return launch_status();
     }
     if (shared > 48 * 1024) {
       cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
       if (err != cudaSuccess) return (int)err;
     }
-    launch_kernel(kernel, dim3(rows), dim3(256), shared, stream, x, delta, dw, w, typed_out, width, eps);
+    launch_kernel(kernel, dim3(rows), dim3(256), shared, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);
     return launch_status();
   };
   if (out_dtype == MLR_F32) return launch(rms_norm_step_kernel<float>, (float*)out);

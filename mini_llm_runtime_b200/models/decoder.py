@@ -88,22 +88,24 @@ class DecoderModel:
     # ------------------------------------------------------------------ forward
     def forward(self, ctx) -> torch.Tensor:
         """Run the step's rows through the model; float32 logits [wanted rows, vocab]."""
-        if self.embedding.needs_positions:
-            residual = self.embedding.forward(ctx.token_ids, ctx.positions)
-        else:
-            residual = self.embedding.forward(ctx.token_ids)
+        residual = self._embed(ctx)
+        # the stream is updated in place: a model that adds the embedding's rows again looks them up a second time
+        embedded = self._embed(ctx) if any(step.add_embedding for step in self.spec.run_order) else None
         pending = None
         for step in self.spec.run_order:
             view = ctx.cache_view(step.cache)
             block = self.blocks[step.layer]
-            if step.offset_row is None:
+            # what is added to the stream before the layer: a vector of the offset table, or the embedding's rows
+            offset = embedded if step.add_embedding else (
+                None if step.offset_row is None else self.offsets.vector(step.offset_row))
+            if offset is None:
                 residual, pending = block.forward(residual, pending, ctx, view, step.writes_cache)
-            elif block.takes_offset:
-                residual, pending = block.forward(residual, pending, ctx, view, step.writes_cache,
-                                                  offset=self.offsets.vector(step.offset_row))
+            elif block.takes_row_offset if step.add_embedding else block.takes_offset:
+                residual, pending = block.forward(residual, pending, ctx, view, step.writes_cache, offset=offset)
             else:
                 residual = self._settle(residual, pending)
-                residual = ctx.ops.add_rows(residual, self.offsets.vector(step.offset_row))
+                residual = (ctx.ops.add_inplace(residual, offset) if step.add_embedding
+                            else ctx.ops.add_rows(residual, offset))
                 residual, pending = block.forward(residual, None, ctx, view, step.writes_cache)
         if ctx.num_wanted == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=residual.device)
@@ -120,6 +122,11 @@ class DecoderModel:
             normed = (self.final_norm.add_forward(rows, delta) if post is None
                       else self.final_norm.add_forward(rows, delta, post=post))
         return self.head.forward(normed, self.embedding)
+
+    def _embed(self, ctx) -> torch.Tensor:
+        if self.embedding.needs_positions:
+            return self.embedding.forward(ctx.token_ids, ctx.positions)
+        return self.embedding.forward(ctx.token_ids)
 
     @staticmethod
     def _settle(residual, pending):

@@ -53,6 +53,8 @@ LIBRARIES: dict[str, tuple[str, ...]] = {
     "attention_sigmoid": (),
     "attention_sigmoid_mma": (),
     "state_space": (),
+    "delta_rule": (),
+    "attention_shaped_mma": (),
 }
 
 _loaded: dict[str, ctypes.CDLL] = {}

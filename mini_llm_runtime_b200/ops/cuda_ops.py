@@ -1337,8 +1337,9 @@ class CudaOps:
         return chosen, weights
 
     def routed_experts(self, x: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, gate_up: torch.Tensor,
-                       down: torch.Tensor, block: int, activation: str = "silu") -> torch.Tensor:
-        """sum_t weights[r, t] * down_e(act(gate_e x_r) * up_e x_r), e = chosen[r, t], as float32 [rows, N].
+                       down: torch.Tensor, block: int, activation: str = "silu", weigh_input: bool = False) -> torch.Tensor:
+        """sum_t weights[r, t] * down_e(act(gate_e x_r) * up_e x_r), e = chosen[r, t], as float32 [rows, N]; with
+        ``weigh_input`` the weight multiplies the expert's input instead: sum_t expert_e(weights[r, t] x_r).
         ``gate_up`` [experts, 2 * inner, K] holds blocks of ``block`` gate rows followed by the up rows
         of the same outputs, ``down`` [experts, N, inner]."""
         _need(x, "x", dims=2)
@@ -1360,16 +1361,17 @@ class CudaOps:
             return out
         lib = build.load_library("routed_experts")
         pairs = rows * top
+        in_weights, out_weights = (weights, None) if weigh_input else (None, weights)
         grouped = (self.use_tensor_cores and self.use_grouped_experts and x.dtype == torch.bfloat16
                    and rows > self.GROUPED_EXPERT_ROWS and K % 8 == 0 and inner % 8 == 0
                    and x.data_ptr() % 16 == 0 and gate_up.data_ptr() % 16 == 0 and down.data_ptr() % 16 == 0)
         if not grouped:
             # every (row, chosen expert) pair streams its expert's matrices
             hidden = torch.empty((pairs, inner), dtype=x.dtype, device=x.device)
-            _check(lib.mlr_expert_hidden(_ptr(x), _ptr(chosen), _ptr(gate_up), _ptr(hidden), rows, K, inner, top,
-                                         int(block), act, _code(x.dtype), _stream()), "expert_hidden")
-            _check(lib.mlr_expert_down(_ptr(hidden), _ptr(chosen), _ptr(weights), _ptr(down), _ptr(out), rows, N, inner,
-                                       top, _code(x.dtype), _stream()), "expert_down")
+            _check(lib.mlr_expert_hidden(_ptr(x), _ptr(chosen), _ptr(in_weights), _ptr(gate_up), _ptr(hidden), rows, K,
+                                         inner, top, int(block), act, _code(x.dtype), _stream()), "expert_hidden")
+            _check(lib.mlr_expert_down(_ptr(hidden), _ptr(chosen), _ptr(out_weights), _ptr(down), _ptr(out), rows, N,
+                                       inner, top, _code(x.dtype), _stream()), "expert_down")
             return out
         # many rows: the pairs sorted by expert, each expert's rows through the tensor-core product with
         # its own matrices (tiles of 128 rows of one expert), the results summed per row in the order
@@ -1382,8 +1384,10 @@ class CudaOps:
         place = torch.empty(pairs, dtype=torch.int32, device=x.device)
         token_of = torch.empty(pairs, dtype=torch.int32, device=x.device)
         tiles = torch.empty(max_tiles * 3, dtype=torch.int32, device=x.device)
-        _check(lib.mlr_sort_pairs(_ptr(chosen), _ptr(place), _ptr(token_of), _ptr(tiles), pairs, top, experts,
-                                  tile_rows, max_tiles, _stream()), "sort_pairs")
+        # weights of the inputs, in the order of the sorted rows: the gate/up product's epilogue applies them
+        row_scale = torch.empty(pairs, dtype=torch.float32, device=x.device) if weigh_input else None
+        _check(lib.mlr_sort_pairs(_ptr(chosen), _ptr(in_weights), _ptr(place), _ptr(token_of), _ptr(row_scale), _ptr(tiles),
+                                  pairs, top, experts, tile_rows, max_tiles, _stream()), "sort_pairs")
         sorted_x = torch.empty((pairs, K), dtype=x.dtype, device=x.device)
         _check(lib.mlr_gather_rows_by(_ptr(x), _ptr(token_of), _ptr(sorted_x), pairs, K * x.element_size(),
                                       _stream()), "gather_rows_by")
@@ -1393,31 +1397,40 @@ class CudaOps:
         if fused:
             hidden = torch.empty((pairs, inner), dtype=x.dtype, device=x.device)
             _check(gemm.mlr_gemm_tcgen05_grouped(_ptr(sorted_x), _ptr(gate_up), _ptr(hidden), _ptr(tiles), max_tiles,
-                                                 pairs, experts, 2 * inner, K, 0, 1 + act, tile_rows, error_word, _stream()),
+                                                 pairs, experts, 2 * inner, K, 0, 1 + act, tile_rows, _ptr(row_scale), error_word,
+                                                 _stream()),
                    "grouped gate/up product")
         else:
             both = torch.empty((pairs, 2 * inner), dtype=x.dtype, device=x.device)
             _check(gemm.mlr_gemm_tcgen05_grouped(_ptr(sorted_x), _ptr(gate_up), _ptr(both), _ptr(tiles), max_tiles,
-                                                 pairs, experts, 2 * inner, K, 0, 0, tile_rows, error_word, _stream()),
+                                                 pairs, experts, 2 * inner, K, 0, 0, tile_rows, _ptr(row_scale), error_word,
+                                                 _stream()),
                    "grouped gate/up product")
             hidden = self.gated_activation(both, block, activation)
         y = torch.empty((pairs, N), dtype=torch.float32, device=x.device)
         _check(gemm.mlr_gemm_tcgen05_grouped(_ptr(hidden), _ptr(down), _ptr(y), _ptr(tiles), max_tiles, pairs, experts,
-                                             N, inner, 1, 0, tile_rows, error_word, _stream()), "grouped down product")
-        _check(lib.mlr_combine_pairs(_ptr(y), _ptr(place), _ptr(weights), _ptr(out), rows, N, top, _stream()),
+                                             N, inner, 1, 0, tile_rows, _ptr(None), error_word, _stream()), "grouped down product")
+        _check(lib.mlr_combine_pairs(_ptr(y), _ptr(place), _ptr(out_weights), _ptr(out), rows, N, top, _stream()),
                "combine_pairs")
         return out
 
     # ------------------------------------------------------------------ 32-bit stream with RMS norms behind the sublayers
     def rms_norm_step(self, x: torch.Tensor, eps: float, *, delta: torch.Tensor | None = None,
                       delta_weight: torch.Tensor | None = None, norm_weight: torch.Tensor | None = None,
-                      out_dtype: torch.dtype | None = None):
+                      out_dtype: torch.dtype | None = None, groups: int = 1, offset: torch.Tensor | None = None):
         """One pass over the rows of the float32 stream ``x`` [rows, width]: x += delta / rms(delta) *
-        delta_weight (when ``delta``, float32, is given), then, with ``out_dtype``, returns x / rms(x) *
-        norm_weight in that dtype, or the rows of x as they are in that dtype when ``norm_weight`` is None.
-        rms(v) = sqrt(mean(v^2) + eps)."""
+        delta_weight (when ``delta``, float32, is given), x += offset (when given: float32, a vector [width] or
+        rows [rows, width]), then, with ``out_dtype``, returns x / rms(x) * norm_weight in that dtype, or the
+        rows of x as they are in that dtype when ``norm_weight`` is None.  rms(v) = sqrt(mean(v^2) + eps), taken
+        over each of ``groups`` equal parts of the row."""
         _need(x, "x", torch.float32, 2)
         rows, width = x.shape
+        if groups <= 0 or width % groups:
+            raise KernelError("the norm's parts must divide the row")
+        if offset is not None:
+            _need(offset, "offset", torch.float32)
+            if tuple(offset.shape) not in ((width,), (rows, width)):
+                raise KernelError("the offset is a vector of the stream's width, or rows of its shape")
         for name, vector in (("delta_weight", delta_weight), ("norm_weight", norm_weight)):
             if vector is not None:
                 _need(vector, name, torch.float32, 1)
@@ -1428,11 +1441,12 @@ class CudaOps:
             if delta.shape != x.shape or delta_weight is None:
                 raise KernelError("delta needs the stream's shape and its norm's weight")
         out = None if out_dtype is None else torch.empty((rows, width), dtype=out_dtype, device=x.device)
-        if delta is None and out is None:
+        if delta is None and out is None and offset is None:
             return None
         _check(build.load_library("stream32").mlr_rms_norm_step(
-            _ptr(x), _ptr(delta), _ptr(delta_weight), _ptr(norm_weight), _ptr(out), rows, width, ctypes.c_float(eps),
-            _code(out_dtype or torch.float32), _stream()), "rms_norm_step")
+            _ptr(x), _ptr(delta), _ptr(delta_weight), _ptr(offset), int(offset is not None and offset.dim() == 2),
+            _ptr(norm_weight), _ptr(out), rows, width, int(groups), ctypes.c_float(eps), _code(out_dtype or torch.float32),
+            _stream()), "rms_norm_step")
         return out
 
     def normed_mean(self, a: torch.Tensor, a_weight: torch.Tensor, b: torch.Tensor, b_weight: torch.Tensor, eps: float,
@@ -1558,6 +1572,151 @@ class CudaOps:
             _ptr(batch.block_table), _ptr(batch.seg_slot), batch.block_table.shape[1], tiles, rows, heads, kv_heads, dim,
             vdim, k_pool.shape[2], ctypes.c_float(scale), _ptr(r1), _ptr(r2), _ptr(score_bias), _ptr(head_mix), chunks,
             max(chunk_keys, 32), _code(q.dtype), _stream()), "sigmoid attention")
+        return out
+
+    # ------------------------------------------------------------------ softmax attention with shaped scores
+    SHAPED_CHUNK_TILES = 4      # key tiles (of 32 keys) a CTA of the tensor-core decode kernel takes at least
+
+    def shaped_attention(self, q: torch.Tensor, key: torch.Tensor, value: torch.Tensor | None, slots: torch.Tensor,
+                         k_pool: torch.Tensor, v_pool: torch.Tensor, batch: AttentionBatch, heads: int, kv_heads: int,
+                         dim: int, vdim: int, scale: float, *, softcap: float = 0.0, slopes: torch.Tensor | None = None,
+                         window: int = 0, chunk: int = 0, sink: torch.Tensor | None = None,
+                         gate: torch.Tensor | None = None, write_kv: bool = True) -> torch.Tensor:
+        """Store the rows' keys (and values) at ``slots`` of the pools, then causal softmax attention with
+        score x = softcap * tanh(q . k * scale / softcap) (q . k * scale without a cap) - slopes_h * (i - j); position
+        i sees the keys j <= i of its own chunk of ``chunk`` positions (0: no chunks) and of its last ``window``
+        positions (0: all); exp(sink_h) joins each head's denominator; the result is multiplied by
+        sigmoid(gate).  q [rows, heads*dim], key [rows, kv_heads*dim], value [rows, kv_heads*vdim] or None (the
+        keys are the values: nothing else is cached), gate [rows, heads*vdim] or None: views with unit column
+        stride in the pools' dtype; slopes, sink: float32 [heads]."""
+        rows = q.shape[0]
+        _need(k_pool, "k_pool", None, 4)
+        dtype = k_pool.dtype
+        for name, view, width in (("q", q, heads * dim), ("key", key, kv_heads * dim), ("value", value, kv_heads * vdim),
+                                  ("gate", gate, heads * vdim)):
+            if view is not None and (not view.is_cuda or view.dtype != dtype or tuple(view.shape) != (rows, width)
+                                     or view.stride(1) != 1):
+                raise KernelError(f"{name} must be a CUDA view [{rows}, {width}] of {dtype} with unit column stride")
+        _need(slots, "slots", torch.int64, 1)
+        for name, vector in (("slopes", slopes), ("sink", sink)):
+            if vector is not None:
+                _need(vector, name, torch.float32, 1)
+                if vector.shape[0] != heads:
+                    raise KernelError(f"{name}: one number per head")
+        if slots.shape[0] != rows or k_pool.shape[1] != kv_heads or k_pool.shape[3] != dim:
+            raise KernelError("one slot per row; the key pool must match the head count and size")
+        shared = value is None
+        if shared:
+            if vdim != dim:
+                raise KernelError("keys that are values have one size")
+            v_pool = k_pool
+        else:
+            _need(v_pool, "v_pool", dtype, 4)
+            if v_pool.shape[:3] != k_pool.shape[:3] or v_pool.shape[3] != vdim:
+                raise KernelError("the value pool does not match the value size")
+        if "tile_seg" not in batch.plan:
+            raise KernelError("the batch carries no attention work lists (plan_attention)")
+        out = torch.empty((rows, heads * vdim), dtype=dtype, device=q.device)
+        page_size = k_pool.shape[2]
+        on_tensor_cores = (shared and self.use_mma_attention and dtype == torch.bfloat16
+                           and self._shaped_mma_fits(dim)
+                           and all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in (q, key))
+                           and (gate is None or (gate.data_ptr() % 4 == 0 and gate.stride(0) % 2 == 0))
+                           and batch.num_decode * heads <= self.ATTENTION_COUNTERS)
+        only_decode = batch.num_decode == batch.num_segments
+        fused_store = on_tensor_cores and only_decode and write_kv      # the decode kernel stores the new keys itself
+        if write_kv and not fused_store:
+            for rows_in, pool, size in ((key, k_pool, dim), (value, v_pool, vdim)):
+                if rows_in is not None:
+                    _check(build.load_library("elementwise").mlr_store_heads(
+                        _ptr(rows_in), ctypes.c_longlong(rows_in.stride(0)), _ptr(slots), _ptr(pool), rows, kv_heads, size,
+                        page_size, pool.element_size(), _stream()), "store_heads")
+        segments = (_ptr(batch.seg_q_start), _ptr(batch.seg_q_len), _ptr(batch.seg_pos0), _ptr(batch.block_table),
+                    _ptr(batch.seg_slot), batch.block_table.shape[1])
+        gate_view = (_ptr(gate), ctypes.c_longlong(0 if gate is None else gate.stride(0)))
+        q_view = (_ptr(q), ctypes.c_longlong(q.stride(0)))
+        if not on_tensor_cores:
+            if batch.counts["tiles"] > 0:
+                _check(build.load_library("attention_generic").mlr_attention_generic_shaped(
+                    *q_view, _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(batch.plan["tile_seg"]),
+                    _ptr(batch.plan["tile_row0"]), *segments, batch.counts["tiles"], heads, kv_heads, dim, vdim, page_size,
+                    int(window), ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(slopes), _ptr(sink), int(chunk),
+                    *gate_view, _code(dtype), _stream()), "shaped attention")
+            return out
+        lib = build.load_library("attention_shaped_mma")
+
+        def launch(decode, fresh, lists, count, partial, counters, splits, what):
+            _check(lib.mlr_attention_shaped_mma(
+                int(decode), *q_view, _ptr(fresh), ctypes.c_longlong(0 if fresh is None else fresh.stride(0)), _ptr(slots),
+                _ptr(k_pool), _ptr(out), *gate_view, _ptr(slopes), _ptr(sink), *lists, count, *segments, heads, kv_heads, dim,
+                page_size, int(window), int(chunk), ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(partial),
+                _ptr(counters), splits, _stream()), what)
+
+        if batch.num_decode > 0:
+            # keys over CTAs so that the step's CTAs fill the device about twice, at least four tiles each
+            longest = min(n for n in (int(batch.max_kv_len), int(window) or 1 << 30, int(chunk) or 1 << 30))
+            tiles = longest // 32 + 2
+            groups = batch.num_decode * kv_heads * -(-(heads // kv_heads) // 16)
+            splits = max(1, min(-(-tiles // self.SHAPED_CHUNK_TILES), 2 * self.sm_count(q.device) // groups, 64))
+            partial = counters = None
+            if splits > 1:
+                partial = torch.empty(batch.num_decode * splits * heads * (dim + 2), dtype=torch.float32, device=q.device)
+                counters = self._workspace(q.device)["attention_counters"]
+            launch(True, key if fused_store else None, (_ptr(None if only_decode else batch.plan["decode_seg"]), _ptr(None)),
+                   batch.num_decode, partial, counters, splits, "shaped attention (decode)")
+        if batch.counts["wide"] > 0:
+            launch(False, None, (_ptr(batch.plan["wide_tile_seg"]), _ptr(batch.plan["wide_tile_row0"])),
+                   batch.counts["wide"], None, None, 1, "shaped attention (prefill)")
+        return out
+
+    def _shaped_mma_fits(self, dim: int) -> bool:
+        cache = self.__dict__.setdefault("_shaped_fits", {})
+        if dim not in cache:
+            cache[dim] = bool(build.load_library("attention_shaped_mma").mlr_attention_shaped_mma_fits(dim))
+        return cache[dim]
+
+    # ------------------------------------------------------------------ gated delta rule
+    def delta_rule_scan(self, q, k, v, a, b, dt_bias, A_log, state, ctx, heads: int, kv_heads: int, dim: int, vdim: int,
+                        unit_eps: float) -> torch.Tensor:
+        """Per request and head h (q and k of head h // (heads / kv_heads)), token after token: u_t = beta_t (v_t -
+        g_t S_{t-1}^T k^_t), S_t = g_t S_{t-1} + k^_t u_t^T, y_t = S_t^T q^_t, with k^ = k / sqrt(sum k^2 + unit_eps), q^ likewise times
+        dim^-0.5, g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b).  q, k [rows, kv_heads*dim], v
+        [rows, heads*vdim], a, b [rows, heads]: float32 views with unit column stride; state: float32 [slots,
+        heads, vdim, dim] (the transposed S), advanced in place; returns float32 [rows, heads*vdim]."""
+        rows = q.shape[0]
+        for name, vector in (("dt_bias", dt_bias), ("A_log", A_log)):
+            _need(vector, name, torch.float32, 1)
+            if vector.shape[0] != heads:
+                raise KernelError(f"{name} needs one entry per head")
+        _need(state, "state", torch.float32, 4)
+        if tuple(state.shape[1:]) != (heads, vdim, dim):
+            raise KernelError(f"state has shape {tuple(state.shape)}, expected [slots, {heads}, {vdim}, {dim}]")
+        y = torch.empty((rows, heads * vdim), dtype=torch.float32, device=q.device)
+        # steps with longer segments take four tokens at once; a first kernel leaves their inner products here
+        coef = torch.empty((rows, heads, 12), dtype=torch.float32, device=q.device) if ctx.max_q_len > 1 else None
+        _check(build.load_library("delta_rule").mlr_delta_rule_scan(
+            *self._view(q, "q", rows, kv_heads * dim), *self._view(k, "k", rows, kv_heads * dim),
+            *self._view(v, "v", rows, heads * vdim), *self._view(a, "a", rows, heads), *self._view(b, "b", rows, heads),
+            _ptr(dt_bias), _ptr(A_log), _ptr(coef), _ptr(state), _ptr(y), _ptr(ctx.seg_q_start), _ptr(ctx.seg_q_len),
+            _ptr(ctx.seg_slot), ctx.num_segments, int(ctx.max_q_len), heads, kv_heads, dim, vdim, ctypes.c_float(unit_eps),
+            ctypes.c_float(float(dim) ** -0.5), _stream()), "delta_rule_scan")
+        return y
+
+    def gated_head_norm(self, y: torch.Tensor, gate, weight: torch.Tensor, eps: float, heads: int,
+                        out_dtype: torch.dtype) -> torch.Tensor:
+        """y / rms(y) * weight * silu(gate) head by head (rms over the head's entries, eps inside the root).
+        y: float32 [rows, heads*vdim]; weight: float32 [vdim], shared by the heads; gate: a float32 view of y's
+        shape, or None for no gate."""
+        _need(y, "y", torch.float32, 2)
+        _need(weight, "weight", torch.float32, 1)
+        rows, inner = y.shape
+        if weight.shape[0] * heads != inner:
+            raise KernelError("gated_head_norm: one weight per entry of a head")
+        gate_view = (ctypes.c_void_p(0), ctypes.c_longlong(0)) if gate is None else self._view(gate, "gate", rows, inner)
+        out = torch.empty((rows, inner), dtype=out_dtype, device=y.device)
+        _check(build.load_library("sequence_mix").mlr_gated_head_norm(
+            _ptr(y), *gate_view, _ptr(weight), _ptr(out), rows, heads, inner // heads, ctypes.c_float(eps),
+            _code(out_dtype), _stream()), "gated_head_norm")
         return out
 
     # ------------------------------------------------------------------ state-space mixer

@@ -18,10 +18,32 @@ from ..ops import AttentionBatch
 from .base import KVCacheNeed, Mixer, TensorSpec, build_part, register_part
 
 
-class GQAAttention(Mixer):
+class PagedAttention(Mixer):
+    """What every mixer over the paged cache shares: the attention kernels' work lists (one set per step for all
+    of them) and the step's ragged batch as the kernels want it."""
+
     graph_safe = True
-    supports_norm_fusion = True
     plan_key = "paged_attention"     # every attention layer of a model reads the same work lists
+
+    def step_plan(self, host):
+        return ops.current().plan_attention(host.lengths, host.position_start)
+
+    def _batch(self, ctx, view) -> AttentionBatch:
+        """The step's ragged batch as the attention kernels want it; built once per step and cache
+        group and shared by the layers of that group."""
+        batch = view.shared.get("attention_batch")
+        if batch is None:
+            arrays, counts = ctx.plans.get(self.plan_key, ({}, {}))
+            batch = AttentionBatch(
+                seg_q_start=ctx.seg_q_start, seg_q_len=ctx.seg_q_len, seg_pos0=ctx.seg_pos0, seg_slot=ctx.seg_slot,
+                block_table=view.block_table, num_segments=ctx.num_segments, max_q_len=ctx.max_q_len,
+                max_kv_len=ctx.max_kv_len, plan=arrays, counts=counts)
+            view.shared["attention_batch"] = batch
+        return batch
+
+
+class GQAAttention(PagedAttention):
+    supports_norm_fusion = True
 
     def __init__(self, spec, compute_dtype):
         super().__init__(spec, compute_dtype)
@@ -86,22 +108,6 @@ class GQAAttention(Mixer):
         self.w_qkv = folded.to(self.compute_dtype).contiguous()
         self.input_norm_eps = float(eps)
 
-    def step_plan(self, host):
-        return ops.current().plan_attention(host.lengths, host.position_start)
-
-    def _batch(self, ctx, view) -> AttentionBatch:
-        """The step's ragged batch as the attention kernels want it; built once per step and cache
-        group and shared by the layers of that group."""
-        batch = view.shared.get("attention_batch")
-        if batch is None:
-            arrays, counts = ctx.plans.get(self.plan_key, ({}, {}))
-            batch = AttentionBatch(
-                seg_q_start=ctx.seg_q_start, seg_q_len=ctx.seg_q_len, seg_pos0=ctx.seg_pos0, seg_slot=ctx.seg_slot,
-                block_table=view.block_table, num_segments=ctx.num_segments, max_q_len=ctx.max_q_len,
-                max_kv_len=ctx.max_kv_len, plan=arrays, counts=counts)
-            view.shared["attention_batch"] = batch
-        return batch
-
     def forward(self, x, ctx, view, writes_cache, raw_input=False, residual=None):
         """``raw_input``: x is the un-normalised stream and the q/k/v product applies the row scale
         of the folded norm.  ``residual``: the output product adds into it in place."""
@@ -122,7 +128,7 @@ class GQAAttention(Mixer):
         return k.linear(mixed, self.w_o, self.b_o, residual=residual)
 
 
-class DifferentialAttention(Mixer):
+class DifferentialAttention(PagedAttention):
     """Grouped-query attention with two softmax maps per head over shared values.
 
     q = Wq x holds, per head, [map 1 | map 2] (2 * dim numbers); k = Wk x likewise per kv head; v = Wv x
@@ -132,9 +138,6 @@ class DifferentialAttention(Mixer):
     a1, a2 the maps' outputs and lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (one number per
     layer): o = a1 - lambda a2, o / rms(o) * (1 - diff), then Wo.  Scores, softmax and norms are
     32-bit; the cache holds normalised keys (both maps side by side) and values."""
-
-    graph_safe = True
-    plan_key = "paged_attention"
 
     def __init__(self, spec, compute_dtype):
         super().__init__(spec, compute_dtype)
@@ -176,20 +179,6 @@ class DifferentialAttention(Mixer):
         l = {n: tensors[p + n].float() for n in ("lq1", "lk1", "lq2", "lk2")}
         self.lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + self.diff
 
-    def step_plan(self, host):
-        return ops.current().plan_attention(host.lengths, host.position_start)
-
-    def _batch(self, ctx, view) -> AttentionBatch:
-        batch = view.shared.get("attention_batch")
-        if batch is None:
-            arrays, counts = ctx.plans.get(self.plan_key, ({}, {}))
-            batch = AttentionBatch(
-                seg_q_start=ctx.seg_q_start, seg_q_len=ctx.seg_q_len, seg_pos0=ctx.seg_pos0, seg_slot=ctx.seg_slot,
-                block_table=view.block_table, num_segments=ctx.num_segments, max_q_len=ctx.max_q_len,
-                max_kv_len=ctx.max_kv_len, plan=arrays, counts=counts)
-            view.shared["attention_batch"] = batch
-        return batch
-
     def forward(self, x, ctx, view, writes_cache):
         k = ops.current()
         qkv = k.linear(x, self.w_qkv, out_dtype=torch.float32)
@@ -201,7 +190,7 @@ class DifferentialAttention(Mixer):
         return k.linear(mixed, self.w_o, out_dtype=torch.float32)
 
 
-class RotatedValueAttention(Mixer):
+class RotatedValueAttention(PagedAttention):
     """Grouped-query softmax attention over all earlier keys, with norms on q, k and v and a rotation
     of the values.
 
@@ -219,9 +208,6 @@ class RotatedValueAttention(Mixer):
 
     32-bit: the norms, angles and rotations, scores and softmax; the projections leave 32-bit rows.
     In bfloat16 the products' operands, q, and the cached keys and values are bfloat16."""
-
-    graph_safe = True
-    plan_key = "paged_attention"
 
     def __init__(self, spec, compute_dtype):
         super().__init__(spec, compute_dtype)
@@ -278,20 +264,6 @@ class RotatedValueAttention(Mixer):
         if self.value_position is not None:
             self.value_position.load({}, device)
 
-    def step_plan(self, host):
-        return ops.current().plan_attention(host.lengths, host.position_start)
-
-    def _batch(self, ctx, view) -> AttentionBatch:
-        batch = view.shared.get("attention_batch")
-        if batch is None:
-            arrays, counts = ctx.plans.get(self.plan_key, ({}, {}))
-            batch = AttentionBatch(
-                seg_q_start=ctx.seg_q_start, seg_q_len=ctx.seg_q_len, seg_pos0=ctx.seg_pos0, seg_slot=ctx.seg_slot,
-                block_table=view.block_table, num_segments=ctx.num_segments, max_q_len=ctx.max_q_len,
-                max_kv_len=ctx.max_kv_len, plan=arrays, counts=counts)
-            view.shared["attention_batch"] = batch
-        return batch
-
     def forward(self, x, ctx, view, writes_cache):
         k = ops.current()
         interleaved = self.position.interleaved
@@ -308,7 +280,7 @@ class RotatedValueAttention(Mixer):
         return k.linear(mixed, self.w_o, out_dtype=torch.float32)
 
 
-class HeadNormAttention(Mixer):
+class HeadNormAttention(PagedAttention):
     """Grouped-query causal attention without a rotation, with q and k RMS-normalised per head.
 
     q = Wq x + bq [heads * dim], k = Wk x + bk [kv_heads * dim], v = Wv x + bv [kv_heads * vdim] (one fused
@@ -331,9 +303,6 @@ class HeadNormAttention(Mixer):
 
     32-bit: the projections' results, the norms, the blend, scores and weights.  In bfloat16 the products'
     operands, q, and the cached keys and values are bfloat16."""
-
-    graph_safe = True
-    plan_key = "paged_attention"
 
     def __init__(self, spec, compute_dtype):
         super().__init__(spec, compute_dtype)
@@ -409,20 +378,6 @@ class HeadNormAttention(Mixer):
         if self.value_mix == "blend":
             self.mix = f32("vmix").reshape(1)
 
-    def step_plan(self, host):
-        return ops.current().plan_attention(host.lengths, host.position_start)
-
-    def _batch(self, ctx, view) -> AttentionBatch:
-        batch = view.shared.get("attention_batch")
-        if batch is None:
-            arrays, counts = ctx.plans.get(self.plan_key, ({}, {}))
-            batch = AttentionBatch(
-                seg_q_start=ctx.seg_q_start, seg_q_len=ctx.seg_q_len, seg_pos0=ctx.seg_pos0, seg_slot=ctx.seg_slot,
-                block_table=view.block_table, num_segments=ctx.num_segments, max_q_len=ctx.max_q_len,
-                max_kv_len=ctx.max_kv_len, plan=arrays, counts=counts)
-            view.shared["attention_batch"] = batch
-        return batch
-
     def forward(self, x, ctx, view, writes_cache):
         k = ops.current()
         qkv = k.linear(x, self.w_qkv, self.b_qkv, out_dtype=torch.float32)
@@ -448,7 +403,90 @@ class HeadNormAttention(Mixer):
         return k.linear(mixed, self.w_o, out_dtype=torch.float32)
 
 
+class ShapedAttention(PagedAttention):
+    """Grouped-query causal softmax attention without a rotation, whose scores are bent and limited by optional
+    pieces that other designs can combine.
+
+    q = Wq x [heads * dim], k = Wk x [kv_heads * dim], v = Wv x [kv_heads * vdim], no biases;
+    ``keys_are_values``: v = k as projected, there is no Wv and only keys are cached.  Query head h reads
+    key/value head h // (heads / kv_heads).  score = (q . k) * ``scale``; ``softcap`` c > 0: score <- c tanh(score /
+    c); ``slopes`` (a number per head): slope_h * (i - j) off the score; ``chunk`` n > 0: position i sees only
+    its own chunk of n positions (counted from the request's start), ``window`` n > 0: only its last n; ``sink``:
+    exp(sink_h), a learned number per head, joins the softmax's denominator; ``gate``: the concatenated heads are
+    multiplied by sigmoid(Wg x) before Wo.
+
+    32-bit: scores, cap, bias, softmax and the sums over keys.  In bfloat16 the projections, the cached keys and
+    values, the gate's projection and the attention's output are bfloat16."""
+
+    def __init__(self, spec, compute_dtype):
+        super().__init__(spec, compute_dtype)
+        a = self.args
+        self.hidden_size = int(a["hidden_size"])
+        self.heads = int(a["heads"])
+        self.kv_heads = int(a.get("kv_heads", self.heads))
+        self.dim = int(a["dim"])
+        self.keys_are_values = bool(a.get("keys_are_values", False))
+        self.vdim = int(a.get("vdim", self.dim))
+        self.scale = float(a["scale"])
+        self.softcap = float(a.get("softcap") or 0.0)
+        self.chunk = int(a.get("chunk") or 0)
+        self.window = int(a.get("window") or 0)
+        self.has_sink = bool(a.get("sink", False))
+        self.has_gate = bool(a.get("gate", False))
+        self.slope_values = a.get("slopes")
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be divisible by kv_heads")
+        if self.keys_are_values and self.vdim != self.dim:
+            raise ValueError("keys that are values have one size")
+        if self.slope_values is not None and len(self.slope_values) != self.heads:
+            raise ValueError("one distance slope per head")
+        self.w_in = self.w_o = self.sink = self.slopes = None
+
+    def cache_need(self):
+        value_dim = 0 if self.keys_are_values else (None if self.vdim == self.dim else self.vdim)
+        return KVCacheNeed(self.kv_heads, self.dim, self.window or None, value_dim=value_dim, chunk=self.chunk or None)
+
+    def _sizes(self):
+        sizes = {"q": self.heads * self.dim, "k": self.kv_heads * self.dim}
+        if not self.keys_are_values:
+            sizes["v"] = self.kv_heads * self.vdim
+        if self.has_gate:
+            sizes["g"] = self.heads * self.vdim
+        return sizes
+
+    def tensors(self):
+        p, h = self.prefix, self.hidden_size
+        out = {p + name: TensorSpec((rows, h)) for name, rows in self._sizes().items()}
+        out[p + "o"] = TensorSpec((h, self.heads * self.vdim))
+        if self.has_sink:
+            out[p + "sink"] = TensorSpec((self.heads,), init="bias")
+        return out
+
+    def load(self, tensors, device):
+        p = self.prefix
+        self.w_in = self._to_compute(torch.cat([tensors[p + name] for name in self._sizes()], dim=0), device)
+        self.w_o = self._to_compute(tensors[p + "o"], device)
+        if self.has_sink:
+            self.sink = tensors[p + "sink"].to(device=device, dtype=torch.float32).contiguous()
+        if self.slope_values is not None:
+            self.slopes = torch.tensor(self.slope_values, dtype=torch.float32, device=device)
+
+    def forward(self, x, ctx, view, writes_cache):
+        k = ops.current()
+        projected = k.linear(x, self.w_in)
+        parts, at = {}, 0
+        for name, width in self._sizes().items():
+            parts[name] = projected[:, at:at + width]
+            at += width
+        mixed = k.shaped_attention(parts["q"], parts["k"], parts.get("v"), view.slots, view.k_pool, view.v_pool,
+                                   self._batch(ctx, view), self.heads, self.kv_heads, self.dim, self.vdim, self.scale,
+                                   softcap=self.softcap, slopes=self.slopes, window=self.window, chunk=self.chunk,
+                                   sink=self.sink, gate=parts.get("g"), write_kv=writes_cache)
+        return k.linear(mixed, self.w_o, out_dtype=torch.float32)
+
+
 register_part("mixer", "gqa_attention", GQAAttention)
+register_part("mixer", "shaped_attention", ShapedAttention)
 register_part("mixer", "head_norm_attention", HeadNormAttention)
 register_part("mixer", "differential_attention", DifferentialAttention)
 register_part("mixer", "rotated_value_attention", RotatedValueAttention)

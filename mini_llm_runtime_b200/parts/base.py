@@ -52,13 +52,30 @@ class TensorSpec:
 class KVCacheNeed:
     """The mixer wants keys and values of its past positions: all of them, or a window.  With a
     window, the first ``keep_first`` positions stay visible (and cached) for the request's whole
-    life.  ``value_dim`` is the size of a value head where it differs from a key head's."""
+    life.  With a ``chunk`` a position sees only its own chunk of so many positions, counted from the
+    request's start.  ``value_dim`` is the size of a value head where it differs from a key head's."""
 
     num_kv_heads: int
     head_dim: int
     window: int | None = None
     value_dim: int | None = None      # 0: no values are stored (a mixer whose values are part of its key rows)
     keep_first: int = 0
+    chunk: int | None = None
+
+    @property
+    def span(self) -> int | None:
+        """Most positions visible at once beside the kept ones; None: all of them."""
+        limits = [n for n in (self.window, self.chunk) if n is not None]
+        return min(limits) if limits else None
+
+    def lowest_visible(self, position: int) -> int:
+        """The lowest position (beside the kept ones) that a query at ``position`` or later can see."""
+        lowest = 0
+        if self.window is not None:
+            lowest = max(lowest, position - self.window + 1)
+        if self.chunk is not None:
+            lowest = max(lowest, position // self.chunk * self.chunk)
+        return lowest
 
     @property
     def value_head_dim(self) -> int:
@@ -265,6 +282,8 @@ class Block:
     # True: ``forward`` accepts ``offset=`` (a vector to add to the stream before the layer) and
     # fuses the add into its first norm; otherwise the model adds the vector itself
     takes_offset = False
+    # True: ``offset=`` may also be a whole tensor of rows [rows, width] (the embedding's)
+    takes_row_offset = False
 
     def forward(self, residual: torch.Tensor, pending, ctx, view,
                 writes_cache: bool) -> tuple[torch.Tensor, "torch.Tensor | PendingDelta | None"]:

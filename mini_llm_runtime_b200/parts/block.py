@@ -81,12 +81,16 @@ class SandwichNorm(Block):
     The stream x is 32-bit floats; the sublayers hand back 32-bit rows.  Each "add the normalised
     output, then norm for the next sublayer" is one pass over the stream: the last output of the
     layer travels on as a ``PendingDelta`` and is added by the next layer's first norm (or the
-    model's final norm), together with a vector the run order may ask to be added before the layer."""
+    model's final norm), together with the vector (or the rows, where the norms take them) that the run order
+    may ask to be added before the layer."""
 
     takes_offset = True
 
+    @property
+    def takes_row_offset(self):
+        return getattr(self.mixer_norm, "adds_rows", False)
+
     def forward(self, residual, pending, ctx, view, writes_cache, offset=None):
-        kernels = ops.current()
         if pending is None:
             normed = self.mixer_norm.forward(residual, offset=offset)
         elif isinstance(pending, PendingDelta):

@@ -14,6 +14,9 @@ Per token, with h the input row:
     out += shared(h)                          with ``shared`` = the inner width of one more gated expert of the
                                               same form that every token uses (tensors ``shared.gate|up|down``)
 
+With ``weigh="input"`` a chosen expert's weight multiplies its input instead of its output: the sum is over
+expert_e(s_e h).
+
 Experts have no biases.  Checkpoint names after the prefix: ``router`` [experts, hidden], ``correction``
 [experts] (``correction=False``: none), ``e<j>.gate``, ``e<j>.up`` [inner, hidden], ``e<j>.down`` [hidden,
 inner].  The experts' matrices are stacked at load time: [experts, 2 * inner, hidden] with gate and up
@@ -55,6 +58,9 @@ class RoutedExperts(FeedForward):
         self.group_top = int(a.get("group_top", 1))
         if self.group_top < 1:
             raise ValueError("a group's score sums at least one choice score")
+        self.weigh = str(a.get("weigh", "output"))
+        if self.weigh not in ("output", "input"):
+            raise ValueError(f"unknown place of the experts' weights {self.weigh!r}; known: output, input")
         self.shared = None
         if a.get("shared"):
             self.shared = build_part("feed_forward", PartSpec("gated_mlp", {
@@ -101,7 +107,8 @@ class RoutedExperts(FeedForward):
         chosen, weights = k.route_experts(x, self.router, self.correction, self.top, self.groups, self.keep,
                                           self.scoring, self.renormalise, group_top=self.group_top,
                                           renorm_eps=self.renorm_eps)
-        out = k.routed_experts(x, chosen, weights, self.w_gate_up, self.w_down, self.block, self.activation)
+        out = k.routed_experts(x, chosen, weights, self.w_gate_up, self.w_down, self.block, self.activation,
+                               weigh_input=self.weigh == "input")
         if self.shared is not None:
             out = k.add_residual(out, self.shared.forward(x, ctx))
         return out

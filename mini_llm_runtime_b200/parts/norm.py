@@ -129,17 +129,21 @@ class LayerNorm(Norm):
 
 class StreamRMSNorm(Norm):
     """RMS norm for a 32-bit residual stream: y = v / sqrt(mean(v^2) + eps) * w, statistics and weight in
-    32-bit.  With ``one_plus`` the checkpoint stores the weight's offset from one: w = 1 + stored.  The
-    checkpoint name comes from the spec (``tensor``).  Uses, each one pass over the stream:
+    32-bit.  With ``one_plus`` the checkpoint stores the weight's offset from one: w = 1 + stored.  With
+    ``groups`` the row is cut into that many equal parts, each divided by its own root mean square.  A
+    ``multiplier`` (of a norm behind a sublayer: how much of it enters the stream) is taken into the weight
+    at load time.  The checkpoint name comes from the spec (``tensor``).  Uses, each one pass over the stream:
 
     * ``forward(x)``: the normalised rows in the compute dtype;
     * ``add_into(stream, delta)``: stream += norm(delta), for a norm that sits behind a sublayer;
     * ``add_cast(stream, delta)``: the same, and the new rows of the stream in the compute dtype (the input
       of a sublayer that reads the stream itself);
-    * ``add_forward(stream, delta, post=)``: stream += post(delta) (``post`` another norm of this kind; the
-      plain delta without one), then this norm of the new stream."""
+    * ``add_forward(stream, delta, post=, offset=)``: stream += post(delta) (``post`` another norm of this
+      kind; the plain delta without one), stream += offset (a vector or rows, if given), then this norm of the
+      new stream."""
 
     graph_safe = True
+    adds_rows = True
 
     def __init__(self, spec, compute_dtype):
         super().__init__(spec, compute_dtype)
@@ -147,6 +151,10 @@ class StreamRMSNorm(Norm):
         self.eps = float(self.args["eps"])
         self.tensor = self.args.get("tensor") or self.prefix + "weight"
         self.one_plus = bool(self.args.get("one_plus", False))
+        self.groups = int(self.args.get("groups", 1))
+        self.multiplier = float(self.args.get("multiplier", 1.0))
+        if self.groups < 1 or self.size % self.groups:
+            raise ValueError("the norm's parts must divide the row")
         self.weight: torch.Tensor | None = None
 
     def tensors(self):
@@ -154,30 +162,33 @@ class StreamRMSNorm(Norm):
 
     def load(self, tensors, device):
         weight = tensors[self.tensor].to(device=device, dtype=torch.float32)
-        self.weight = (1.0 + weight if self.one_plus else weight).contiguous()
+        weight = 1.0 + weight if self.one_plus else weight
+        self.weight = (weight if self.multiplier == 1.0 else weight * self.multiplier).contiguous()
 
-    def forward(self, x):
-        return ops.current().rms_norm_step(x, self.eps, norm_weight=self.weight, out_dtype=self.compute_dtype)
+    def forward(self, x, offset=None):
+        return ops.current().rms_norm_step(x, self.eps, norm_weight=self.weight, out_dtype=self.compute_dtype,
+                                           groups=self.groups, offset=offset)
 
     def add_into(self, stream, delta):
-        ops.current().rms_norm_step(stream, self.eps, delta=delta, delta_weight=self.weight)
+        ops.current().rms_norm_step(stream, self.eps, delta=delta, delta_weight=self.weight, groups=self.groups)
         return stream
 
     def add_cast(self, stream, delta):
         if self.compute_dtype == torch.float32:
             return self.add_into(stream, delta)
         return ops.current().rms_norm_step(stream, self.eps, delta=delta, delta_weight=self.weight,
-                                           out_dtype=self.compute_dtype)
+                                           out_dtype=self.compute_dtype, groups=self.groups)
 
-    def add_forward(self, residual, delta, post=None):
+    def add_forward(self, residual, delta, post=None, offset=None):
         if post is None:
             ops.current().add_residual(residual, delta)
-            return self.forward(residual)
-        if post.eps != self.eps:
+            return self.forward(residual, offset)
+        if post.eps != self.eps or getattr(post, "groups", 1) != self.groups:
             post.add_into(residual, delta)
-            return self.forward(residual)
+            return self.forward(residual, offset)
         return ops.current().rms_norm_step(residual, self.eps, delta=delta, delta_weight=post.weight,
-                                           norm_weight=self.weight, out_dtype=self.compute_dtype)
+                                           norm_weight=self.weight, out_dtype=self.compute_dtype, groups=self.groups,
+                                           offset=offset)
 
 
 register_part("norm", "rms_norm", RMSNorm)

@@ -12,6 +12,7 @@ recurrence; the mixer's output projection leaves 32-bit rows for a 32-bit residu
            out = Wo (o / rms(o) * norm * silu(Wg x_g)).
 ``state_space``  a selective state-space layer with a scalar decay per head (Mamba-2, "state-space
            duality"), see ``StateSpaceMixer``.
+``gated_delta_rule``  a delta rule with a scalar decay and step size per head, see ``DeltaRuleMixer``.
 ``hgrn2``  gated linear attention whose forget gate also sets what is written:
            f_t = l + (1 - l) sigmoid(Wf x + b);  S <- diag(f_t) S + (1 - f_t) v_t^T;
            o_t = S^T silu(Wq x);  out = Wo (o / rms(o) * norm).
@@ -207,6 +208,84 @@ class StateSpaceMixer(Mixer):
         return k.linear(gated, self.w_o, out_dtype=torch.float32)
 
 
+class DeltaRuleMixer(Mixer):
+    """Gated delta rule: a recurrence that writes, per head and token, the difference between the value and
+    what the state already answers to the key.
+
+    q = Wq x and k = Wk x [kv_heads * dim], v = Wv x [heads * vdim] each pass a causal convolution per channel
+    (``<name>.conv`` [channels, taps], last column the current token's, zeros before the request's start) and
+    silu; head h reads the q and k of head h // (heads / kv_heads).  k and q are divided by sqrt(sum of squares
+    + ``unit_eps``), q also multiplied by dim^-0.5.  Per head g = exp(-exp(A_log) softplus(Wa x + dt_bias)),
+    beta = sigmoid(Wb x) and, on a state S [dim, vdim],
+    S_t = g_t S_{t-1} + k_t u_t^T with u_t = beta_t (v_t - g_t S_{t-1}^T k_t), and o_t = S_t^T q_t.
+    Every head's o is divided by its root mean square over vdim, times ``norm`` [vdim] (shared by the heads),
+    times silu(Wg x); then Wo.
+
+    Per request the layer carries S (32-bit, kept transposed: [heads, vdim, dim]) and the convolution's last
+    taps - 1 inputs.  Everything between the projections and Wo is 32-bit."""
+
+    graph_safe = True
+
+    def __init__(self, spec, compute_dtype):
+        super().__init__(spec, compute_dtype)
+        a = self.args
+        self.hidden_size = int(a["hidden_size"])
+        self.heads = int(a["heads"])
+        self.kv_heads = int(a.get("kv_heads", self.heads))
+        self.dim = int(a["dim"])
+        self.vdim = int(a["vdim"])
+        self.taps = int(a["conv"])
+        self.eps = float(a["eps"])
+        self.unit_eps = float(a["unit_eps"])
+        if self.heads % self.kv_heads or self.taps < 1:
+            raise ValueError("heads must be divisible by kv_heads, and the convolution needs at least one tap")
+        self.qk, self.inner = self.kv_heads * self.dim, self.heads * self.vdim
+        self.channels = 2 * self.qk + self.inner
+        self.w_in = self.w_o = self.conv = self.dt_bias = self.a_log = self.norm = None
+
+    def cache_need(self):
+        return (StateNeed((self.heads, self.vdim, self.dim), torch.float32, "state"),
+                StateNeed((self.taps - 1, self.channels), torch.float32, "conv"))
+
+    def tensors(self):
+        p, h = self.prefix, self.hidden_size
+        sizes = {"q": self.qk, "k": self.qk, "v": self.inner}
+        out = {p + name: TensorSpec((rows, h)) for name, rows in sizes.items()}
+        out.update({p + name + ".conv": TensorSpec((rows, self.taps), init="bias") for name, rows in sizes.items()})
+        out.update({p + "g": TensorSpec((self.inner, h)), p + "a": TensorSpec((self.heads, h)),
+                    p + "b": TensorSpec((self.heads, h)), p + "A_log": TensorSpec((self.heads,), init="bias"),
+                    p + "dt_bias": TensorSpec((self.heads,), init="bias"),
+                    p + "norm": TensorSpec((self.vdim,), init="norm"), p + "o": TensorSpec((h, self.inner))})
+        return out
+
+    def load(self, tensors, device):
+        p = self.prefix
+        # one product yields [q | k | v | g | a | b], filled up with zeros so that its rows start at 16-byte boundaries
+        rows = [tensors[p + name] for name in ("q", "k", "v", "g", "a", "b")]
+        fill = -(2 * self.inner + 2 * self.qk + 2 * self.heads) % 8
+        if fill:
+            rows.append(torch.zeros((fill, self.hidden_size), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = self._to_compute(torch.cat(rows, dim=0), device)
+        self.w_o = self._to_compute(tensors[p + "o"], device)
+        self.conv = _float(torch.cat([tensors[p + name + ".conv"] for name in "qkv"], dim=0), device)
+        self.dt_bias = _float(tensors[p + "dt_bias"], device)
+        self.a_log = _float(tensors[p + "A_log"], device)
+        self.norm = _float(tensors[p + "norm"], device)
+
+    def forward(self, x, ctx, view, writes_cache):
+        k = ops.current()
+        qk, channels, inner = self.qk, self.channels, self.inner
+        projected = k.linear(x, self.w_in, out_dtype=torch.float32)
+        mixed = k.causal_conv(projected[:, :channels], self.conv, None, view.states["conv"], ctx, "silu")
+        at = channels + inner
+        y = k.delta_rule_scan(mixed[:, :qk], mixed[:, qk:2 * qk], mixed[:, 2 * qk:], projected[:, at:at + self.heads],
+                              projected[:, at + self.heads:at + 2 * self.heads], self.dt_bias, self.a_log,
+                              view.states["state"], ctx, self.heads, self.kv_heads, self.dim, self.vdim, self.unit_eps)
+        gated = k.gated_head_norm(y, projected[:, channels:at], self.norm, self.eps, self.heads, self.compute_dtype)
+        return k.linear(gated, self.w_o, out_dtype=torch.float32)
+
+
 register_part("mixer", "wkv", WKVMixer)
+register_part("mixer", "gated_delta_rule", DeltaRuleMixer)
 register_part("mixer", "state_space", StateSpaceMixer)
 register_part("mixer", "hgrn2", HGRN2Mixer)

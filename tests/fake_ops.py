@@ -444,13 +444,16 @@ class FakeOps:
             weights = weights / (weights.sum(-1, keepdim=True) + renorm_eps)
         return chosen.to(torch.int32), weights
 
-    def routed_experts(self, x, chosen, weights, gate_up, down, block, activation="silu"):
+    def routed_experts(self, x, chosen, weights, gate_up, down, block, activation="silu", weigh_input=False):
         out = torch.zeros((x.shape[0], down.shape[1]), dtype=torch.float32)
         for row in range(x.shape[0]):
             for t in range(chosen.shape[1]):
                 e = int(chosen[row, t])
-                hidden = self.gated_activation(self.linear(x[row:row + 1], gate_up[e]), block, activation)
-                out[row] += weights[row, t] * (hidden.float() @ down[e].float().T)[0]
+                product = self.linear(x[row:row + 1], gate_up[e])
+                if weigh_input:
+                    product = product * weights[row, t]
+                hidden = self.gated_activation(product, block, activation)
+                out[row] += (1.0 if weigh_input else weights[row, t]) * (hidden.float() @ down[e].float().T)[0]
         return out
 
     # ---- 32-bit stream with RMS norms behind the sublayers
@@ -458,12 +461,18 @@ class FakeOps:
     def _rms(v, eps):
         return v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps)
 
-    def rms_norm_step(self, x, eps, *, delta=None, delta_weight=None, norm_weight=None, out_dtype=None):
+    def rms_norm_step(self, x, eps, *, delta=None, delta_weight=None, norm_weight=None, out_dtype=None, groups=1,
+                      offset=None):
+        def rms(v):
+            return self._rms(v.view(v.shape[0], groups, -1), eps).view(v.shape)
+
         if delta is not None:
-            x += self._rms(delta, eps) * delta_weight
+            x += rms(delta) * delta_weight
+        if offset is not None:
+            x += offset
         if out_dtype is None:
             return None
-        return (x.clone() if norm_weight is None else self._rms(x, eps) * norm_weight).to(out_dtype)
+        return (x.clone() if norm_weight is None else rms(x) * norm_weight).to(out_dtype)
 
     def normed_mean(self, a, a_weight, b, b_weight, eps, factor):
         return factor * (self._rms(a, eps) * a_weight + self._rms(b, eps) * b_weight)
@@ -535,8 +544,78 @@ class FakeOps:
             for tap in range(taps):
                 total = total + padded[tap:tap + segment.length] * weight[:, tap]
             out[rows] = torch.nn.functional.silu(total) if activation == "silu" else total
-            state[segment.slot] = padded[-(taps - 1):]
+            if taps > 1:
+                state[segment.slot] = padded[-(taps - 1):]
         return out
+
+    # ---- softmax attention with shaped scores; gated delta rule
+    def shaped_attention(self, q, key, value, slots, k_pool, v_pool, batch, heads, kv_heads, dim, vdim, scale, *, softcap=0.0,
+                         slopes=None, window=0, chunk=0, sink=None, gate=None, write_kv=True):
+        rows, page_size, group = q.shape[0], k_pool.shape[2], heads // kv_heads
+        if write_kv:
+            for source, pool in ((key, k_pool), (value, v_pool)):
+                if source is None:
+                    continue
+                for t in range(rows):
+                    slot = int(slots[t])
+                    if slot >= 0:
+                        page, offset = divmod(slot, page_size)
+                        pool[page, :, offset, :] = source[t].reshape(kv_heads, -1)
+        if value is None:
+            v_pool = k_pool
+        out = torch.empty((rows, heads * vdim), dtype=q.dtype)
+        q3 = q.float().reshape(rows, heads, dim)
+        for seg in range(batch.num_segments):
+            start, length, pos0 = int(batch.seg_q_start[seg]), int(batch.seg_q_len[seg]), int(batch.seg_pos0[seg])
+            table = batch.block_table[int(batch.seg_slot[seg])]
+            for r in range(length):
+                p = pos0 + r
+                lowest = max(p // chunk * chunk if chunk else 0, p - window + 1 if window else 0)
+                keys = torch.arange(lowest, p + 1)
+                pages = table[(keys // page_size).long()].long()
+                assert (pages >= 0).all(), "attention reads a page the request does not hold"
+                offsets = (keys % page_size).long()
+                k = k_pool[pages, :, offsets, :].float().repeat_interleave(group, dim=1)
+                v = v_pool[pages, :, offsets, :].float().repeat_interleave(group, dim=1)
+                scores = torch.einsum("hd,khd->hk", q3[start + r], k) * scale
+                if softcap:
+                    scores = softcap * torch.tanh(scores / softcap)
+                if slopes is not None:
+                    scores = scores - slopes[:, None] * (p - keys).float()[None, :]
+                if sink is not None:
+                    scores = torch.cat([scores, sink[:, None]], dim=1)
+                weights = torch.softmax(scores, dim=-1)[:, :len(keys)]
+                mixed = torch.einsum("hk,khd->hd", weights, v).reshape(-1)
+                if gate is not None:
+                    mixed = mixed * torch.sigmoid(gate[start + r].float())
+                out[start + r] = mixed.to(q.dtype)
+        return out
+
+    def delta_rule_scan(self, q, k, v, a, b, dt_bias, A_log, state, ctx, heads, kv_heads, dim, vdim, unit_eps):
+        def unit(x):
+            x = x.reshape(-1, kv_heads, dim)
+            return (x * torch.rsqrt((x * x).sum(-1, keepdim=True) + unit_eps)).repeat_interleave(heads // kv_heads, dim=1)
+
+        kn, qn = unit(k), unit(q) * dim ** -0.5
+        decay = torch.exp(-torch.exp(A_log) * torch.nn.functional.softplus(a + dt_bias))
+        beta = torch.sigmoid(b)
+        y = torch.empty((q.shape[0], heads * vdim), dtype=torch.float32)
+        for segment in ctx.segments:
+            S = state[segment.slot]                   # [heads, vdim, dim]
+            for row in range(segment.row_start, segment.row_start + segment.length):
+                S = decay[row].view(heads, 1, 1) * S
+                u = beta[row][:, None] * (v[row].view(heads, vdim) - torch.einsum("hvd,hd->hv", S, kn[row]))
+                S = S + u[:, :, None] * kn[row][:, None, :]
+                y[row] = torch.einsum("hvd,hd->hv", S, qn[row]).reshape(-1)
+            state[segment.slot] = S
+        return y
+
+    def gated_head_norm(self, y, gate, weight, eps, heads, out_dtype):
+        rows = y.shape[0]
+        v = (self._rms(y.reshape(rows, heads, -1), eps) * weight).reshape(y.shape)
+        if gate is not None:
+            v = v * torch.nn.functional.silu(gate)
+        return v.to(out_dtype)
 
     def state_space_scan(self, x, B, C, dt_raw, dt_bias, A_log, D, state, ctx, heads, vdim, n, groups):
         y = torch.empty((x.shape[0], heads * vdim), dtype=torch.float32)
