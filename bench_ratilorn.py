@@ -34,7 +34,7 @@ def ratilorn_config(size):
     s = SIZES[size]
     heads = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5}
     right = {**s["ssm"], "groups": 1, "conv": TAPS, "norm_groups": 1}
-    mlp = {"kind": "moe", "expert": {"ff": s["ff"]}, "shared": {"ff": s["shared"]},
+    mlp = {"kind": "moe", "expert": {"ff": s["ff"]}, **({"shared": {"ff": s["shared"]}} if s["shared"] else {}),
            "router": {"experts": s["experts"], "top": s["top"],
                       "groups": {"count": s["router_groups"][0], "keep": s["router_groups"][1]}}}
     group = [{"type": "parallel", "mixer": {"left": heads, "right": right}, "mlp": mlp},

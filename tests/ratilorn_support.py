@@ -215,13 +215,16 @@ class REngine:
         self.device = device
         self.config = config_from_dict(config_dict)
         self.model = build_model(self.config, dtype)
-        self.tensors = draw_tensors(self.model.expected_tensors(), seed, overrides)
+        self.tensors = self.draw(self.model.expected_tensors(), seed, overrides)
         self.model.load(self.tensors, device)
         self.cache = CacheManager(self.model.cache_needs(), page_size=page_size, num_pages=num_pages,
                                   max_requests=max_requests, max_tokens_per_request=max_tokens, dtype=dtype,
                                   device=device, max_step_tokens=max_step_tokens or max_tokens)
         self.runner = ModelRunner(self.model, self.cache)
         self.runner.graph_capture_after = 1
+
+    def draw(self, expected, seed, overrides):
+        return draw_tensors(expected, seed, overrides)
 
     def plain(self, tokens, config_dict=None, tensors=None):
         return plain_logits(config_dict or self.config_dict, tensors or self.tensors, tokens)
