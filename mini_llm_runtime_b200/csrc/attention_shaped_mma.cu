@@ -23,6 +23,13 @@ namespace mlr {
 
 constexpr float LOG2E = 1.4426950408889634f;
 
+// 2^x by the hardware's approximate instruction (about 2 ulp); minus infinity gives 0.
+__device__ __forceinline__ float exp2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 struct ShapedArgs {
   const bf16* q; long long q_stride;             // rows of heads * D
   const bf16* fresh; long long fresh_stride;     // decode: rows of kv_heads * D with the new keys, or null (already cached)
@@ -37,7 +44,7 @@ struct ShapedArgs {
   int table_width, heads, kv_heads, page_size, page_shift, window, chunk;
   float in_scale, out_scale;                     // capped: scale / cap and cap * log2(e); else scale * log2(e) and 1
   int capped;
-  float* partial; int* counters; int splits;     // decode
+  float* partial; float2* limits; int* counters; int splits;     // decode
 };
 
 // tanh of every number of a fragment.  Small arguments (the usual case by far: a cap is chosen well above the
@@ -105,14 +112,14 @@ __device__ __forceinline__ void shaped_softmax_step(float (*s)[4], float (*o)[4]
     tile_max[i] = fmaxf(tile_max[i], __shfl_xor_sync(0xffffffffu, tile_max[i], 2));
     const float m_new = fmaxf(m[i], tile_max[i]);
     base[i] = m_new == -INFINITY ? 0.f : m_new;       // nothing visible yet: keep everything at zero
-    alpha[i] = exp2f(m[i] - base[i]);                 // m = -inf gives 0
+    alpha[i] = exp2_approx(m[i] - base[i]);                 // m = -inf gives 0
     m[i] = m_new;
   }
 #pragma unroll
   for (int j = 0; j < NT; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      s[j][e] = exp2f(s[j][e] - base[e >> 1]);
+      s[j][e] = exp2_approx(s[j][e] - base[e >> 1]);
       row_sum[e >> 1] += s[j][e];
     }
 #pragma unroll
@@ -183,7 +190,7 @@ __device__ __forceinline__ int lowest_visible(const ShapedArgs& p, int position)
 }
 
 template <int D>
-__global__ void __launch_bounds__(ATTN_THREADS)
+__global__ void __launch_bounds__(ATTN_THREADS, D <= 64 ? 4 : 3)
 shaped_prefill_kernel(const ShapedArgs p) {
   pdl_trigger();
   pdl_wait();
@@ -284,8 +291,8 @@ shaped_prefill_kernel(const ShapedArgs p) {
     if (r >= rows) continue;
     float factor = 1.f / l[i];
     if (p.sinks != nullptr) {
-      const float sink = p.sinks[head] * LOG2E, top = fmaxf(m[i], sink), share = exp2f(m[i] - top);
-      factor = share / fmaf(l[i], share, exp2f(sink - top));
+      const float sink = p.sinks[head] * LOG2E, top = fmaxf(m[i], sink), share = exp2_approx(m[i] - top);
+      factor = share / fmaf(l[i], share, exp2_approx(sink - top));
     }
     const size_t row = (size_t)(q_start + row0 + r);
     const int column = head * D + (lane & 3) * 2;
@@ -308,6 +315,7 @@ shaped_prefill_kernel(const ShapedArgs p) {
 constexpr int DEC_KEYS = 32;         // keys of a warp's tile
 constexpr int DEC_STAGES = 2;
 constexpr int DEC_ROWS = 16;         // query heads of one CTA
+constexpr int DEC_MAX_SPLITS = 64;
 constexpr int DEC_MIN_TILES = 4;     // key tiles a CTA takes at least (one per warp)
 
 // grid: (items, kv heads * blocks of 16 query heads, splits)
@@ -432,8 +440,8 @@ shaped_decode_kernel(const ShapedArgs p) {
   auto finish = [&](float value, float top, float total, int head, int d) {
     float factor = 1.f / total;
     if (p.sinks != nullptr) {
-      const float sink = p.sinks[head] * LOG2E, high = fmaxf(top, sink), part = exp2f(top - high);
-      factor = part / fmaf(total, part, exp2f(sink - high));
+      const float sink = p.sinks[head] * LOG2E, high = fmaxf(top, sink), part = exp2_approx(top - high);
+      factor = part / fmaf(total, part, exp2_approx(sink - high));
     }
     value *= factor;
     if (p.gate != nullptr) {
@@ -450,19 +458,16 @@ shaped_decode_kernel(const ShapedArgs p) {
     float value = 0.f, total = 0.f;
 #pragma unroll
     for (int w = 0; w < ATTN_WARPS; ++w) {
-      const float part = warp_max_[w][r] == -INFINITY ? 0.f : exp2f(warp_max_[w][r] - top);
+      const float part = warp_max_[w][r] == -INFINITY ? 0.f : exp2_approx(warp_max_[w][r] - top);
       value = fmaf(merged[(w * DEC_ROWS + r) * D + d], part, value);
       total = fmaf(warp_sum_[w][r], part, total);
     }
     if (p.splits == 1) {
       finish(value, top, total, head0 + r, d);
     } else {
-      float* dst = p.partial + (((size_t)item * p.splits + blockIdx.z) * p.heads + head0 + r) * (D + 2);
-      dst[d] = value;
-      if (d == 0) {
-        dst[D] = top;
-        dst[D + 1] = total;
-      }
+      const size_t part = ((size_t)item * p.splits + blockIdx.z) * p.heads + head0 + r;
+      p.partial[part * D + d] = value;
+      if (d == 0) p.limits[part] = make_float2(top, total);
     }
   }
   if (p.splits == 1) return;
@@ -476,22 +481,49 @@ shaped_decode_kernel(const ShapedArgs p) {
   if (!is_last) return;
   __threadfence();
   if (threadIdx.x == 0) *counter = 0;
-  const size_t step = (size_t)p.heads * (D + 2);
-  for (int idx = threadIdx.x; idx < live * D; idx += ATTN_THREADS) {
-    const int r = idx / D, d = idx - r * D;
-    const float* src = p.partial + ((size_t)item * p.splits * p.heads + head0 + r) * (D + 2);
+  // a factor per (head, part): the parts' maxima brought together, a warp per head, lanes over the parts
+  float* factors = merged;                                   // [16][splits]
+  const size_t first_part = (size_t)item * p.splits * p.heads + head0;
+  for (int r = warp; r < live; r += ATTN_WARPS) {
+    float2 mine[DEC_MAX_SPLITS / 32];
     float top = -INFINITY;
-#pragma unroll 4
-    for (int z = 0; z < p.splits; ++z) top = fmaxf(top, __ldcg(src + z * step + D));
-    float value = 0.f, total = 0.f;
-#pragma unroll 4
-    for (int z = 0; z < p.splits; ++z) {
-      const float high = __ldcg(src + z * step + D);
-      const float part = high == -INFINITY ? 0.f : exp2f(high - top);
-      value = fmaf(__ldcg(src + z * step + d), part, value);
-      total = fmaf(__ldcg(src + z * step + D + 1), part, total);
+#pragma unroll
+    for (int k = 0; k < DEC_MAX_SPLITS / 32; ++k) {
+      const int z = k * 32 + lane;
+      mine[k] = z < p.splits ? __ldcg(&p.limits[first_part + (size_t)z * p.heads + r]) : make_float2(-INFINITY, 0.f);
+      top = fmaxf(top, mine[k].x);
     }
-    finish(value, top, total, head0 + r, d);
+    top = warp_max(top);
+    float total = 0.f;
+#pragma unroll
+    for (int k = 0; k < DEC_MAX_SPLITS / 32; ++k) {
+      const float part = mine[k].x == -INFINITY ? 0.f : exp2_approx(mine[k].x - top);
+      if (k * 32 + lane < p.splits) factors[r * p.splits + k * 32 + lane] = part;
+      total = fmaf(mine[k].y, part, total);
+    }
+    total = warp_sum(total);
+    if (lane == 0) {
+      warp_max_[0][r] = top;
+      warp_sum_[0][r] = total;
+    }
+  }
+  __syncthreads();
+  for (int idx = threadIdx.x * 4; idx < live * D; idx += ATTN_THREADS * 4) {
+    const int r = idx / D, d = idx - r * D;
+    const float* src = p.partial + (first_part + r) * D + d;
+    const size_t step = (size_t)p.heads * D;
+    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int z = 0; z < p.splits; ++z) {
+      const float4 v = __ldcg(reinterpret_cast<const float4*>(src + z * step));
+      const float part = factors[r * p.splits + z];
+      sum.x = fmaf(v.x, part, sum.x); sum.y = fmaf(v.y, part, sum.y);
+      sum.z = fmaf(v.z, part, sum.z); sum.w = fmaf(v.w, part, sum.w);
+    }
+    finish(sum.x, warp_max_[0][r], warp_sum_[0][r], head0 + r, d);
+    finish(sum.y, warp_max_[0][r], warp_sum_[0][r], head0 + r, d + 1);
+    finish(sum.z, warp_max_[0][r], warp_sum_[0][r], head0 + r, d + 2);
+    finish(sum.w, warp_max_[0][r], warp_sum_[0][r], head0 + r, d + 3);
   }
 }
 
@@ -554,7 +586,7 @@ MLR_EXPORT int mlr_attention_shaped_mma(int decode, const void* q, long long q_s
   if (!aligned(q) || !aligned(fresh) || !aligned(pool) || !aligned(out) || q_stride % 8 || fresh_stride % 8 ||
       gate_stride % 2 || (reinterpret_cast<uintptr_t>(gate) & 3))
     return MLR_BAD_ALIGNMENT;
-  if (heads > 65535 || splits > 65535) return MLR_TOO_LARGE;
+  if (heads > 65535 || splits > DEC_MAX_SPLITS) return MLR_TOO_LARGE;
   ShapedArgs p;
   p.q = (const bf16*)q; p.q_stride = q_stride;
   p.fresh = (const bf16*)fresh; p.fresh_stride = fresh_stride; p.slots = slots;
@@ -571,7 +603,9 @@ MLR_EXPORT int mlr_attention_shaped_mma(int decode, const void* q, long long q_s
   p.capped = softcap > 0.f;
   p.in_scale = p.capped ? scale / softcap : scale * LOG2E;
   p.out_scale = p.capped ? softcap * LOG2E : 1.f;
-  p.partial = partial; p.counters = counters; p.splits = splits;
+  p.partial = partial;                             // the parts, then their maxima and denominators
+  p.limits = partial == nullptr ? nullptr : reinterpret_cast<float2*>(partial + (size_t)count * splits * heads * dim);
+  p.counters = counters; p.splits = splits;
   switch (dim) {
     case 32: return decode ? launch_shaped_decode<32>(p, count, stream) : launch_shaped_prefill<32>(p, count, stream);
     case 64: return decode ? launch_shaped_decode<64>(p, count, stream) : launch_shaped_prefill<64>(p, count, stream);

@@ -29,7 +29,6 @@
 
 namespace mlr {
 
-constexpr int DELTA_THREADS = 128;
 constexpr int DELTA_COEF = 12;
 
 struct DeltaArgs {
@@ -57,7 +56,8 @@ __device__ __forceinline__ float delta_beta(float raw) { return 1.f / (1.f + exp
 constexpr int PREP_WARPS = 4;
 __global__ void __launch_bounds__(PREP_WARPS * 32)
 delta_prepare_kernel(DeltaArgs p) {
-  pdl_trigger();
+  // The recurrence behind this kernel is few blocks that run long: brought in while this kernel's many blocks
+  // still fill the SMs, they would land several to an SM.  So there is no early trigger here.
   pdl_wait();
   const int seg = blockIdx.y, kv = blockIdx.z;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -174,16 +174,16 @@ __device__ __forceinline__ int spread_sums(float (&v)[N], int lane) {
 // lane E key channels of them (in interleaved pieces of four: neighbouring lanes read neighbouring 16-byte
 // pieces of a staged row).  TB tokens per turn; TB == 1 computes its numbers itself.  WIDE: rows are staged
 // in 16-byte pieces (sizes and strides multiples of four floats, pointers aligned).
-template <int E, int SL, int C, int TB, bool WIDE>
-__global__ void __launch_bounds__(DELTA_THREADS)
+template <int E, int SL, int C, int TB, bool WIDE, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 delta_scan_kernel(DeltaArgs p) {
   pdl_trigger();
   extern __shared__ __align__(16) float shared[];
-  constexpr int GROUPS = DELTA_THREADS / SL, COLS = GROUPS * C;
+  constexpr int GROUPS = THREADS / SL, COLS = GROUPS * C;
   constexpr int N = TB * C;
   constexpr int TOKENS = SL == 32 ? 16 : 32;      // tokens staged at once
   const int D = p.dim, V = p.vdim;
-  const int pitch = (D + 3) & ~3;                                     // staged rows are 16-byte aligned
+  constexpr int pitch = E * SL;                                       // staged rows of keys and queries, filled up with zeros
   const int buffer = TOKENS * (2 * pitch + COLS + DELTA_COEF);  // floats of one staging buffer
   const int seg = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS;
   const int kv = head / (p.heads / p.kv_heads);
@@ -192,6 +192,13 @@ delta_scan_kernel(DeltaArgs p) {
   pdl_wait();
   const int q_start = p.seg_q_start[seg], q_len = p.seg_q_len[seg];
 
+  // zeros that no copy overwrites: behind the rows' D entries
+  if (D < pitch) {
+    for (int idx = threadIdx.x; idx < 4 * TOKENS * (pitch - D); idx += THREADS) {
+      const int row = idx / (pitch - D), d = D + idx - row * (pitch - D);
+      shared[(row / (2 * TOKENS)) * buffer + (row % (2 * TOKENS)) * pitch + d] = 0.f;
+    }
+  }
   auto stage = [&](int t0, int which) {
     float* k_rows = shared + which * buffer;
     float* q_rows = k_rows + TOKENS * pitch;
@@ -201,29 +208,29 @@ delta_scan_kernel(DeltaArgs p) {
     const size_t row0 = (size_t)(q_start + t0);
     if (WIDE) {
       const int per_row = D >> 2;
-      for (int idx = threadIdx.x; idx < tokens * per_row; idx += DELTA_THREADS) {
+      for (int idx = threadIdx.x; idx < tokens * per_row; idx += THREADS) {
         const int t = idx / per_row, d = (idx - t * per_row) << 2;
         copy_async_16(k_rows + t * pitch + d, p.k + (row0 + t) * p.k_stride + (size_t)kv * D + d);
         copy_async_16(q_rows + t * pitch + d, p.q + (row0 + t) * p.q_stride + (size_t)kv * D + d);
       }
       constexpr int PIECES = COLS / 4;
-      for (int idx = threadIdx.x; idx < tokens * PIECES; idx += DELTA_THREADS) {
+      for (int idx = threadIdx.x; idx < tokens * PIECES; idx += THREADS) {
         const int t = idx / PIECES, c = (idx - t * PIECES) << 2;
         if (col0 + c < V) copy_async_16(v_rows + t * COLS + c, p.v + (row0 + t) * p.v_stride + (size_t)head * V + col0 + c);
       }
     } else {
-      for (int idx = threadIdx.x; idx < tokens * D; idx += DELTA_THREADS) {
+      for (int idx = threadIdx.x; idx < tokens * D; idx += THREADS) {
         const int t = idx / D, d = idx - t * D;
         copy_async_4(k_rows + t * pitch + d, p.k + (row0 + t) * p.k_stride + (size_t)kv * D + d);
         copy_async_4(q_rows + t * pitch + d, p.q + (row0 + t) * p.q_stride + (size_t)kv * D + d);
       }
-      for (int idx = threadIdx.x; idx < tokens * COLS; idx += DELTA_THREADS) {
+      for (int idx = threadIdx.x; idx < tokens * COLS; idx += THREADS) {
         const int t = idx / COLS, c = idx - t * COLS;
         if (col0 + c < V) copy_async_4(v_rows + idx, p.v + (row0 + t) * p.v_stride + (size_t)head * V + col0 + c);
       }
     }
     if (TB > 1) {
-      for (int idx = threadIdx.x; idx < tokens * 3; idx += DELTA_THREADS) {
+      for (int idx = threadIdx.x; idx < tokens * 3; idx += THREADS) {
         const int t = idx / 3, c = (idx - t * 3) << 2;
         copy_async_16(coef + t * DELTA_COEF + c, p.coef + ((row0 + t) * p.heads + head) * DELTA_COEF + c);
       }
@@ -232,6 +239,15 @@ delta_scan_kernel(DeltaArgs p) {
       copy_async_4(coef + threadIdx.x * DELTA_COEF + 1, p.b + (row0 + threadIdx.x) * p.b_stride + head);
     }
     copy_async_commit();
+    if (TB > 1 && tokens % TB != 0) {      // the rest of the last block of tokens: nothing is read, written or forgotten
+      const int fill = TB - tokens % TB;
+      for (int idx = threadIdx.x; idx < fill * pitch; idx += THREADS) {
+        k_rows[tokens * pitch + idx] = 0.f;
+        q_rows[tokens * pitch + idx] = 0.f;
+      }
+      for (int idx = threadIdx.x; idx < fill * COLS; idx += THREADS) v_rows[tokens * COLS + idx] = 0.f;
+      for (int idx = threadIdx.x; idx < fill * DELTA_COEF; idx += THREADS) coef[tokens * DELTA_COEF + idx] = 0.f;
+    }
   };
 
   stage(0, 0);
@@ -270,7 +286,7 @@ delta_scan_kernel(DeltaArgs p) {
     const float* v_rows = q_rows + TOKENS * pitch;
     float* coef = const_cast<float*>(v_rows) + TOKENS * COLS;
     if (TB == 1) {
-      for (int t = threadIdx.x >> 5; t < tokens; t += DELTA_THREADS / 32) {
+      for (int t = threadIdx.x >> 5; t < tokens; t += THREADS / 32) {
         float kk = 0.f, qq = 0.f, qk = 0.f;
         for (int d = lane; d < D; d += 32) {
           const float kd = k_rows[t * pitch + d], qd = q_rows[t * pitch + d];
@@ -295,74 +311,76 @@ delta_scan_kernel(DeltaArgs p) {
       }
       __syncthreads();
     }
-    for (int t = 0; t < tokens; t += TB) {
-      // the block's dot products with the state before it; the keys stay in registers for the update
-      float kd[TB][E], dk[TB][C], dq[N];
+    // a block's rows are read from shared memory while the block before is worked on
+    float4 k_next[TB][E / 4], q_next[TB][E / 4];
+    auto read_rows = [&](int t) {
 #pragma unroll
       for (int n = 0; n < TB; ++n)
 #pragma unroll
-        for (int c = 0; c < C; ++c) dk[n][c] = dq[n * C + c] = 0.f;
+        for (int i = 0; i < E / 4; ++i) {
+          k_next[n][i] = *reinterpret_cast<const float4*>(k_rows + (t + n) * pitch + entry(4 * i));
+          q_next[n][i] = *reinterpret_cast<const float4*>(q_rows + (t + n) * pitch + entry(4 * i));
+        }
+    };
+    constexpr bool AHEAD = E == 4;      // with more key channels per lane the registers do better otherwise
+    if (AHEAD) read_rows(0);
+    for (int t = 0; t < tokens; t += TB) {
+      // the block's dot products with the state before it; the keys stay in registers for the update
+      if (!AHEAD) read_rows(t);
+      float kd[TB][E], dk[N], dq[N];
 #pragma unroll
-      for (int i = 0; i < E; i += 4) {
-        const bool in = entry(i) < D;
+      for (int n = 0; n < N; ++n) dk[n] = dq[n] = 0.f;
+#pragma unroll
+      for (int n = 0; n < TB; ++n) {
+#pragma unroll
+        for (int i = 0; i < E / 4; ++i) {
+          kd[n][4 * i] = k_next[n][i].x; kd[n][4 * i + 1] = k_next[n][i].y;
+          kd[n][4 * i + 2] = k_next[n][i].z; kd[n][4 * i + 3] = k_next[n][i].w;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < E / 4; ++i) {
 #pragma unroll
         for (int n = 0; n < TB; ++n) {
-          const bool live = in && (TB == 1 || t + n < tokens);
-          float qd[4];
-          if (WIDE) {
-            float4 k4 = make_float4(0.f, 0.f, 0.f, 0.f), q4 = k4;
-            if (live) {
-              k4 = *reinterpret_cast<const float4*>(k_rows + (t + n) * pitch + entry(i));
-              q4 = *reinterpret_cast<const float4*>(q_rows + (t + n) * pitch + entry(i));
-            }
-            kd[n][i] = k4.x; kd[n][i + 1] = k4.y; kd[n][i + 2] = k4.z; kd[n][i + 3] = k4.w;
-            qd[0] = q4.x; qd[1] = q4.y; qd[2] = q4.z; qd[3] = q4.w;
-          } else {
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const bool ok = live && entry(i + j) < D;
-              kd[n][i + j] = ok ? k_rows[(t + n) * pitch + entry(i + j)] : 0.f;
-              qd[j] = ok ? q_rows[(t + n) * pitch + entry(i + j)] : 0.f;
-            }
-          }
+          const float qd[4] = {q_next[n][i].x, q_next[n][i].y, q_next[n][i].z, q_next[n][i].w};
 #pragma unroll
           for (int c = 0; c < C; ++c) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-              dk[n][c] = fmaf(kd[n][i + j], S[c][i + j], dk[n][c]);
-              dq[n * C + c] = fmaf(qd[j], S[c][i + j], dq[n * C + c]);
+              dk[n * C + c] = fmaf(kd[n][4 * i + j], S[c][4 * i + j], dk[n * C + c]);
+              dq[n * C + c] = fmaf(qd[j], S[c][4 * i + j], dq[n * C + c]);
             }
           }
         }
       }
-      // every lane of the group needs the key sums (the u follow from them); the query sums are spread
+      if (AHEAD && t + TB < tokens) read_rows(t + TB);
+      // the key sums are needed by every lane of the group (the u follow from them), the query sums by one
+      if (N <= SL) {
+        spread_sums<N, SL>(dk, lane);
+        const float mine = dk[0];
 #pragma unroll
-      for (int m = SL / 2; m > 0; m >>= 1)
+        for (int n = 0; n < N; ++n) dk[n] = __shfl_sync(0xffffffffu, mine, n * (SL / N), SL);
+      } else {
 #pragma unroll
-        for (int n = 0; n < TB; ++n)
+        for (int m = SL / 2; m > 0; m >>= 1)
 #pragma unroll
-          for (int c = 0; c < C; ++c) dk[n][c] += __shfl_xor_sync(0xffffffffu, dk[n][c], m);
+          for (int n = 0; n < N; ++n) dk[n] += __shfl_xor_sync(0xffffffffu, dk[n], m);
+      }
       const int first = spread_sums<N, SL>(dq, lane);
       float u[TB][C], w[TB], all = 1.f;
 #pragma unroll
       for (int n = 0; n < TB; ++n) {
-        if (TB == 1 || t + n < tokens) {
-          const float4 c0 = *reinterpret_cast<const float4*>(coef + (t + n) * DELTA_COEF);
-          const float4 c1 = *reinterpret_cast<const float4*>(coef + (t + n) * DELTA_COEF + 4);
-          w[n] = c0.w;
-          all = c1.w;
-          const float l[3] = {c1.x, c1.y, c1.z};
+        const float4 c0 = *reinterpret_cast<const float4*>(coef + (t + n) * DELTA_COEF);
+        const float4 c1 = *reinterpret_cast<const float4*>(coef + (t + n) * DELTA_COEF + 4);
+        w[n] = c0.w;
+        if (n == 0) all = c1.w;
+        const float l[3] = {c1.x, c1.y, c1.z};
 #pragma unroll
-          for (int c = 0; c < C; ++c) {
-            float read = c0.x * dk[n][c];
+        for (int c = 0; c < C; ++c) {
+          float read = c0.x * dk[n * C + c];
 #pragma unroll
-            for (int m = 0; m < n; ++m) read = fmaf(l[m < 3 ? m : 0], u[m][c], read);
-            u[n][c] = c0.z * (v_rows[(t + n) * COLS + group * C + c] - read);
-          }
-        } else {
-          w[n] = 0.f;
-#pragma unroll
-          for (int c = 0; c < C; ++c) u[n][c] = 0.f;
+          for (int m = 0; m < n; ++m) read = fmaf(l[m < 3 ? m : 0], u[m][c], read);
+          u[n][c] = c0.z * (v_rows[(t + n) * COLS + group * C + c] - read);
         }
       }
       // this lane's outputs: number `first + i` is token number / C, column number % C
@@ -372,14 +390,16 @@ delta_scan_kernel(DeltaArgs p) {
         for (int i = 0; i < HELD; ++i) {
           const int number = first + i, n = number / C, c = number % C;
           if (t + n < tokens && col0 + group * C + c < V) {
-            const float* mine = coef + (t + n) * DELTA_COEF;
-            float o = mine[1] * dq[i];
+            const float b = coef[(t + n) * DELTA_COEF + 1];
+            const float4 m4 = *reinterpret_cast<const float4*>(coef + (t + n) * DELTA_COEF + 8);      // zero beyond the token
+            const float m[4] = {m4.x, m4.y, m4.z, m4.w};
+            float o = b * dq[i];
 #pragma unroll
-            for (int m = 0; m < TB; ++m) {
-              float um = u[m][0];
+            for (int e = 0; e < TB; ++e) {
+              float ue = u[e][0];
 #pragma unroll
-              for (int cc = 1; cc < C; ++cc) um = c == cc ? u[m][cc] : um;
-              if (m <= n) o = fmaf(mine[8 + m], um, o);
+              for (int cc = 1; cc < C; ++cc) ue = c == cc ? u[e][cc] : ue;
+              o = fmaf(m[e], ue, o);
             }
             p.y[((size_t)(q_start + t0 + t + n) * p.heads + head) * V + col0 + group * C + c] = o;
           }
@@ -418,19 +438,19 @@ delta_scan_kernel(DeltaArgs p) {
   }
 }
 
-template <int E, int SL, int C, int TB, bool WIDE>
+template <int E, int SL, int C, int TB, bool WIDE, int THREADS = 128>
 static int launch_delta(const DeltaArgs& p, int segments, cudaStream_t stream) {
-  constexpr int COLS = DELTA_THREADS / SL * C;
-  const int pitch = (p.dim + 3) & ~3;
+  constexpr int COLS = THREADS / SL * C;
+  constexpr int pitch = E * SL;
   constexpr int TOKENS = SL == 32 ? 16 : 32;
   const size_t shared = sizeof(float) * 2 * (size_t)TOKENS * (2 * pitch + COLS + DELTA_COEF);
   if (shared > 227 * 1024) return MLR_TOO_LARGE;
-  auto kernel = delta_scan_kernel<E, SL, C, TB, WIDE>;
+  auto kernel = delta_scan_kernel<E, SL, C, TB, WIDE, THREADS>;
   if (shared > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     if (err != cudaSuccess) return (int)err;
   }
-  launch_kernel(kernel, dim3(segments, p.heads, (p.vdim + COLS - 1) / COLS), dim3(DELTA_THREADS), shared, stream, p);
+  launch_kernel(kernel, dim3(segments, p.heads, (p.vdim + COLS - 1) / COLS), dim3(THREADS), shared, stream, p);
   return launch_status();
 }
 
@@ -465,10 +485,15 @@ MLR_EXPORT int mlr_delta_rule_scan(const float* q, long long q_stride, const flo
     launch_kernel(delta_prepare_kernel, dim3(blocks, segments, kv_heads), dim3(PREP_WARPS * 32), 0, stream, p);
     const int status = launch_status();
     if (status != MLR_OK) return status;
-    if (dim <= 32) return launch_delta<4, 8, 2, 4, true>(p, segments, stream);
-    if (dim <= 64) return launch_delta<8, 8, 2, 4, true>(p, segments, stream);
-    if (dim <= 128) return launch_delta<16, 8, 2, 4, true>(p, segments, stream);
-    if (dim <= 256) return launch_delta<16, 16, 2, 4, true>(p, segments, stream);
+    if (dim <= 32) return launch_delta<4, 8, 1, 4, true>(p, segments, stream);
+    if (dim <= 64) return launch_delta<4, 16, 1, 4, true>(p, segments, stream);
+    if (dim <= 128) {
+      // one column per group while that many warps still fit the device well, else two (a row read from shared
+      // memory then serves both): 2,048 tokens, 32 heads of 128 x 64: 335 / 398 us, of 128 x 128: 521 / 420 us
+      if ((long long)segments * heads * vdim <= 20LL * sm_count()) return launch_delta<8, 16, 1, 4, true, 256>(p, segments, stream);
+      return launch_delta<8, 16, 2, 4, true>(p, segments, stream);
+    }
+    if (dim <= 256) return launch_delta<8, 32, 2, 4, true>(p, segments, stream);
     return launch_delta<16, 32, 2, 4, true>(p, segments, stream);
   }
   if (wide) {

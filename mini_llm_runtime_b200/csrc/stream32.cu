@@ -200,6 +200,7 @@ layer_norm_step_warp_kernel(float* x, const float* delta, const float* __restric
 template <int THREADS>
 __device__ __forceinline__ float block_sum_of(float v, float* scratch) {
   v = warp_sum(v);
+  if (THREADS == 32) return v;
   __syncthreads();
   if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
   __syncthreads();
@@ -606,12 +607,14 @@ MLR_EXPORT int mlr_rms_norm_step(float* x, const float* delta, const float* dw, 
   const size_t shared = sizeof(float) * ((size_t)width + 32);
   if (shared > 200 * 1024) return MLR_TOO_LARGE;
   auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  const bool few = rows <= 64 * groups && width % 4 == 0 && width <= 8192 && aligned(x) && aligned(delta) && aligned(dw) &&
-                   aligned(offset) && aligned(w) && aligned(out);
+  const bool pieces_fit = width % 4 == 0 && width <= 8192 && aligned(x) && aligned(delta) && aligned(dw) &&
+                          aligned(offset) && aligned(w) && aligned(out);
   auto launch = [&](auto kernel, auto* typed_out) -> int {
     using T = std::remove_pointer_t<decltype(typed_out)>;
-    if (few) {
-      if (width <= 2048)
+    if (pieces_fit) {
+      if (width <= 512 && rows > 1024)      // many small parts: a warp each
+        launch_kernel(rms_norm_step_row_kernel<T, 32>, dim3(rows), dim3(32), 0, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);
+      else if (width <= 2048)
         launch_kernel(rms_norm_step_row_kernel<T, 128>, dim3(rows), dim3(128), 0, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);
       else if (width <= 4096)
         launch_kernel(rms_norm_step_row_kernel<T, 256>, dim3(rows), dim3(256), 0, stream, x, delta, dw, offset, offset_rows, w, typed_out, width, groups, eps);

@@ -276,10 +276,10 @@ def test_prefill_against_token_by_token(name, dtype):
     engine = vs.VEngine(config, dtype, DEVICE, seed=({"MIXED": 14, "ODD": 16, "PLAIN": 1} if dtype == F32 else {"MIXED": 12, "ODD": 8, "PLAIN": 1})[name])
     tokens = vs.tokens_for(config["vocab"], 75, 8)
     want = engine.plain(tokens)
-    # heads of five to ten entries in bfloat16: a rounding weighs more (the stand-in kernels in bfloat16: 0.06)
-    limit = 0.12 if (name, dtype) == ("ODD", BF16) else None
+    # heads of five to ten entries: a rounding weighs more
+    spread = 8e-2 if name == "ODD" else 4e-2
     for what, cuts in (("whole", []), ("token by token", range(1, 75)), ("prompt then decode", [40] + list(range(41, 75)))):
-        vs.assert_logits_close(engine.run_cuts(what, tokens, cuts), want, dtype, what, limit)
+        vs.assert_logits_close(engine.run_cuts(what, tokens, cuts), want, dtype, what, spread)
 
 
 @pytest.mark.parametrize("cuts", [[2, 4, 6, 8], [3, 19, 20, 52], [16, 32, 48, 64], [1, 2, 35, 37, 90], [21, 42, 50, 63]])
