@@ -150,6 +150,91 @@ __device__ __forceinline__ void fa_wait(uint64_t* bar, uint32_t parity, int* err
   if (!gave_up) gave_up = !mbar_wait(bar, parity, error_word, code);
 }
 
+// What bends, limits and weighs the scores beyond scale, causal limit and window (shaped instantiation only):
+// x = cap * tanh(q.k * scale / cap) - slope_h (i - j), keys of the row's own chunk, exp(sink_h) in the
+// denominator, the result times sigmoid(gate).  Everything in powers of two.
+struct FaScore {
+  float in_scale, out_scale;        // capped: scale / cap and cap * log2(e); else scale * log2(e) and 1
+  int capped, chunk;                // chunk 0: none
+  const float *slopes, *sinks;      // [heads] or null
+  const bf16* gate;                 // rows of heads * D, or null
+  long long gate_stride;
+};
+
+// A row's 64 raw scores to shaped ones.  tanh as an odd polynomial in the raw score (its Taylor series): up to
+// the fifth power while all of the warp's arguments are below 0.1, to the ninth below 1/4 (error below 3e-9 of
+// the cap either way), else by the exponential.  The polynomial takes scale, cap and log2(e) into its factors.
+__device__ __forceinline__ void fa_shape_scores(float (&s)[FA_KEYS], const FaScore& f, float slope2, float start) {
+  const float2 step2 = make_float2(slope2, slope2);
+  if (!f.capped) {
+    const float2 a2 = make_float2(f.in_scale, f.in_scale);
+#pragma unroll
+    for (int c = 0; c < FA_KEYS; c += 2) {
+      const float2 bias = __ffma2_rn(step2, make_float2((float)c, (float)(c + 1)), make_float2(start, start));
+      const float2 x = __ffma2_rn(make_float2(s[c], s[c + 1]), a2, bias);
+      s[c] = x.x;
+      s[c + 1] = x.y;
+    }
+    return;
+  }
+  float part[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int c = 0; c < FA_KEYS; c += 8)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) part[e] = fa_max3(part[e], fabsf(s[c + 2 * e]), fabsf(s[c + 2 * e + 1]));
+  const float top = fmaxf(fmaxf(part[0], part[1]), fmaxf(part[2], part[3])) * fabsf(f.in_scale);
+  const float k1 = f.in_scale * f.out_scale, i2 = f.in_scale * f.in_scale;
+  const float k3 = -k1 * i2 * (1.f / 3.f), k5 = k1 * i2 * i2 * (2.f / 15.f);
+  const float2 k1p = make_float2(k1, k1), k3p = make_float2(k3, k3), k5p = make_float2(k5, k5);
+  if (!__any_sync(0xffffffffu, !(top <= 0.1f))) {
+#pragma unroll
+    for (int c = 0; c < FA_KEYS; c += 2) {
+      const float2 v = make_float2(s[c], s[c + 1]), v2 = __fmul2_rn(v, v);
+      const float2 bias = __ffma2_rn(step2, make_float2((float)c, (float)(c + 1)), make_float2(start, start));
+      const float2 x = __ffma2_rn(v, __ffma2_rn(v2, __ffma2_rn(v2, k5p, k3p), k1p), bias);
+      s[c] = x.x;
+      s[c + 1] = x.y;
+    }
+  } else if (!__any_sync(0xffffffffu, !(top <= 0.25f))) {
+    const float k7 = k1 * i2 * i2 * i2 * (-17.f / 315.f), k9 = k1 * i2 * i2 * i2 * i2 * (62.f / 2835.f);
+    const float2 k7p = make_float2(k7, k7), k9p = make_float2(k9, k9);
+#pragma unroll
+    for (int c = 0; c < FA_KEYS; c += 2) {
+      const float2 v = make_float2(s[c], s[c + 1]), v2 = __fmul2_rn(v, v);
+      const float2 bias = __ffma2_rn(step2, make_float2((float)c, (float)(c + 1)), make_float2(start, start));
+      const float2 high = __ffma2_rn(v2, __ffma2_rn(v2, k9p, k7p), k5p);
+      const float2 x = __ffma2_rn(v, __ffma2_rn(v2, __ffma2_rn(v2, high, k3p), k1p), bias);
+      s[c] = x.x;
+      s[c + 1] = x.y;
+    }
+  } else {
+#pragma unroll
+    for (int c = 0; c < FA_KEYS; ++c) {
+      // 1 - 2 / (1 + e^(2|t|)), odd in t; the exponent is kept where the division is defined
+      const float t = s[c] * f.in_scale;
+      const float y = copysignf(1.f - __fdividef(2.f, 1.f + __expf(fminf(2.f * fabsf(t), 80.f))), t);
+      s[c] = fmaf(y, f.out_scale, fmaf(slope2, (float)c, start));
+    }
+  }
+}
+
+// 32 numbers of an output row times sigmoid of the row's gate.
+__device__ __forceinline__ void fa_gate32(float* v, const bf16* gate) {
+#pragma unroll
+  for (int c = 0; c < 32; c += 8) {
+    uint4 raw;      // gate rows start at even columns only: four loads of two
+    const unsigned int* src = reinterpret_cast<const unsigned int*>(gate + c);
+    raw.x = __ldcg(src); raw.y = __ldcg(src + 1); raw.z = __ldcg(src + 2); raw.w = __ldcg(src + 3);
+    const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 g = __bfloat1622float2(pairs[e]);
+      v[c + 2 * e] = __fdividef(v[c + 2 * e], 1.f + __expf(fminf(-g.x, 80.f)));
+      v[c + 2 * e + 1] = __fdividef(v[c + 2 * e + 1], 1.f + __expf(fminf(-g.y, 80.f)));
+    }
+  }
+}
+
 // 32 values of one output row, scaled, as bfloat16 to global memory.
 __device__ __forceinline__ void fa_store32(bf16* dst, const float* v, float factor) {
 #pragma unroll
@@ -164,7 +249,7 @@ __device__ __forceinline__ void fa_store32(bf16* dst, const float* v, float fact
   }
 }
 
-template <int D>
+template <int D, bool SHAPED>
 __global__ void __launch_bounds__(FA_THREADS, 2)      // two CTAs per SM: at most 204 registers
 prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                                  const __grid_constant__ CUtensorMap v_map, bf16* __restrict__ out,
@@ -174,7 +259,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
                                  int table_width, int num_tiles, int heads, int kv_heads, int page_size,
                                  int page_shift, int window, float scale_log2, int* queue, int* error_word,
                                  int max_parts, int tiles_per_unit, float* __restrict__ scratch,
-                                 int* __restrict__ counters, int shared_bytes) {
+                                 int* __restrict__ counters, int shared_bytes, const FaScore score) {
   using Shape = FaShape<D>;
   constexpr int STAGES = Shape::STAGES;
   extern __shared__ uint8_t fa_shared_raw[];
@@ -234,7 +319,12 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
     const int rows = min(FA_ROWS, q_len - row0);
     const int* table = block_table + (size_t)(seg_slot != nullptr ? seg_slot[seg] : seg) * table_width;
     const int first_pos = pos0 + row0, last_pos = first_pos + rows - 1;
-    const int lowest = window > 0 ? max(0, first_pos - window + 1) : 0;
+    // the lowest key a position sees
+    auto lowest_of = [&](int position) {
+      const int lo = window > 0 ? max(0, position - window + 1) : 0;
+      return SHAPED && score.chunk > 0 ? max(lo, position / score.chunk * score.chunk) : lo;
+    };
+    const int lowest = lowest_of(first_pos);
     // An item with many key tiles is cut into parts of equal length; each part is a unit of its
     // own (its state goes to scratch memory, the part that finishes last merges them in part order).
     const int item_begin = lowest / FA_KEYS, item_tiles = last_pos / FA_KEYS - item_begin + 1;
@@ -369,13 +459,14 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
       const int r = threadIdx.x;                                    // row of the item = tensor-memory lane
       const int position = first_pos + r;
       const int limit_hi = r < rows ? position : -1;                // rows past the portion see nothing
-      const int limit_lo = window > 0 ? max(0, position - window + 1) : 0;
+      const int limit_lo = lowest_of(position);
       const uint32_t lane_base = tmem_base + ((uint32_t)(warp * 32) << 16);
       // every row of this warp sees all of a key tile that ends at or before the warp's first
       // position and begins at or after the window start of the warp's last row
       const bool warp_full = warp * 32 + 31 < rows;
       const int warp_first = first_pos + warp * 32;
-      const int warp_lo = window > 0 ? max(0, first_pos + min(rows - 1, warp * 32 + 31) - window + 1) : 0;
+      const int warp_lo = lowest_of(first_pos + min(rows - 1, warp * 32 + 31));
+      const float slope2 = SHAPED && score.slopes != nullptr ? score.slopes[head] * 1.4426950408889634f : 0.f;
       float m_run = -INFINITY;      // the running max of the scaled scores (base-2 exponent)
       float m_base = -INFINITY;     // the exponent that sum, probabilities and output are relative to
       float l = 0.f;
@@ -393,6 +484,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
         fa_tmem_wait_ld();
         fa_fence_before();
 
+        if (SHAPED) fa_shape_scores(s, score, slope2, slope2 * (float)(key0 - position));
         if (!(warp_full && key0 + FA_KEYS - 1 <= warp_first && key0 >= warp_lo)) {
 #pragma unroll
           for (int c = 0; c < FA_KEYS; ++c) {
@@ -504,7 +596,15 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
         // so that the 128 threads write and read neighbouring addresses
         float* states = scratch + (size_t)item * max_parts * STATE * FA_ROWS + r;
         float* mine = states + (size_t)part * STATE * FA_ROWS;
-        const float inv = 1.f / l;
+        // the factor of the finished row: one over the sum, the sink's share included
+        auto finish_factor = [&](float top, float sum) {
+          if (!SHAPED || score.sinks == nullptr) return 1.f / sum;
+          const float sink = score.sinks[head] * 1.4426950408889634f, high = fmaxf(top, sink), share = fa_exp2(top - high);
+          return share / fmaf(sum, share, fa_exp2(sink - high));
+        };
+        const float inv = finish_factor(m_base, l);
+        const bf16* gate = SHAPED && score.gate != nullptr && r < rows
+                               ? score.gate + (size_t)(q_start + row0 + r) * score.gate_stride + (size_t)head * D : nullptr;
         bf16* dst = out + ((size_t)(q_start + row0 + r) * heads + head) * D;
 #pragma unroll
         for (int c = 0; c < D; c += 32) {
@@ -513,6 +613,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
           fa_tmem_load16(lane_base + FA_TMEM_O + c + 16, reinterpret_cast<uint32_t*>(o) + 16);
           fa_tmem_wait_ld();
           if (parts == 1) {
+            if (SHAPED && gate != nullptr) fa_gate32(o, gate + c);
             if (r < rows) fa_store32(dst + c, o, inv);
           } else {
 #pragma unroll
@@ -543,7 +644,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
                   l_all = fmaf(__ldcg(theirs + FA_ROWS), factor[q], l_all);
                 }
               }
-              const float inv_all = 1.f / l_all;
+              const float inv_all = finish_factor(m_all, l_all);
 #pragma unroll
               for (int c = 0; c < D; c += 32) {
                 float o[32];
@@ -557,6 +658,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
                     for (int d = 0; d < 32; ++d) o[d] = fmaf(__ldcg(theirs + d * FA_ROWS), factor[q], o[d]);
                   }
                 }
+                if (SHAPED && gate != nullptr) fa_gate32(o, gate + c);
                 fa_store32(dst + c, o, inv_all);
               }
             }
@@ -602,17 +704,18 @@ static const int units_per_cta = 1;
 
 namespace mlr {
 
-template <int D>
+template <int D, bool SHAPED = false>
 static int fa_launch(const void* q, const void* k_pool, const void* v_pool, void* out, const int* tile_seg,
                      const int* tile_row0, const int* seg_q_start, const int* seg_q_len, const int* seg_pos0,
                      const int* block_table, const int* seg_slot, int table_width, int tiles, int q_rows, int heads,
                      int kv_heads, int page_size, int page_shift, long long pool_rows, int window, float scale,
                      int max_kv_len, int* queue, int* error_word, void* scratch, long long scratch_bytes,
-                     int* counters, int counters_len, cudaStream_t stream) {
+                     int* counters, int counters_len, cudaStream_t stream, long long q_stride = 0,
+                     const FaScore& score = FaScore{}) {
   using Shape = FaShape<D>;
   const int box_rows = page_size >= FA_KEYS ? FA_KEYS : page_size;
   CUtensorMap q_map, k_map, v_map;
-  if (!cached_tile_map(&q_map, q, q_rows, (long long)heads * D, FA_ROWS) ||
+  if (!cached_tile_map(&q_map, q, q_rows, q_stride > 0 ? q_stride : (long long)heads * D, FA_ROWS) ||
       !cached_tile_map(&k_map, k_pool, pool_rows, D, box_rows) ||
       !cached_tile_map(&v_map, v_pool, pool_rows, D, box_rows))
     return MLR_BAD_SIZE;
@@ -622,7 +725,7 @@ static int fa_launch(const void* q, const void* k_pool, const void* v_pool, void
   const size_t shared = (D == 64 ? 1024 : 0) + (size_t)Shape::DATA_BYTES + FA_CONTROL_BYTES;
   static bool configured = false;
   if (!configured) {
-    cudaError_t err = cudaFuncSetAttribute(prefill_attention_tcgen05_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+    cudaError_t err = cudaFuncSetAttribute(prefill_attention_tcgen05_kernel<D, SHAPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     if (err != cudaSuccess) return (int)err;
     configured = true;
   }
@@ -645,10 +748,10 @@ static int fa_launch(const void* q, const void* k_pool, const void* v_pool, void
   }
   const long long units = items * max_parts;
   const int ctas = (int)(units < resident ? units : resident);
-  launch_kernel(prefill_attention_tcgen05_kernel<D>, dim3(ctas), dim3(FA_THREADS), shared, stream, q_map, k_map, v_map,
+  launch_kernel(prefill_attention_tcgen05_kernel<D, SHAPED>, dim3(ctas), dim3(FA_THREADS), shared, stream, q_map, k_map, v_map,
                 (bf16*)out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot, table_width, tiles, heads,
-                kv_heads, page_size, page_shift, window, scale * 1.4426950408889634f, queue, error_word, max_parts,
-                tiles_per_unit, (float*)scratch, counters, (int)shared);
+                kv_heads, page_size, page_shift, window, SHAPED ? 1.f : scale * 1.4426950408889634f, queue, error_word, max_parts,
+                tiles_per_unit, (float*)scratch, counters, (int)shared, score);
   return launch_status();
 }
 
@@ -686,4 +789,49 @@ MLR_EXPORT int mlr_attention_prefill_tcgen05(const void* q, const void* k_pool, 
   return fa_launch<128>(q, k_pool, v_pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table,
                         seg_slot, table_width, tiles, q_rows, heads, kv_heads, page_size, page_shift, pool_rows, window,
                         scale, max_kv_len, queue, error_word, scratch, scratch_bytes, counters, counters_len, stream);
+}
+
+// The same with shaped scores over keys that are also the values (pool: [pool_pages, kv_heads, page_size,
+// head_dim]).  q: rows spaced q_stride apart (a multiple of 8), starting at the row's first column; softcap 0: no
+// cap; slopes, sinks: float32 [heads] or null; chunk, window 0: none; gate: bfloat16 rows of heads * head_dim
+// entries spaced gate_stride apart (even), or null.
+MLR_EXPORT int mlr_attention_shaped_prefill_tcgen05(
+    const void* q, long long q_stride, const void* pool, void* out, const int* tile_seg, const int* tile_row0,
+    const int* seg_q_start, const int* seg_q_len, const int* seg_pos0, const int* block_table, const int* seg_slot,
+    int table_width, int tiles, int q_rows, int heads, int kv_heads, int head_dim, int page_size, int pool_pages, int window,
+    int chunk, float scale, float softcap, const float* slopes, const float* sinks, const void* gate, long long gate_stride,
+    int max_kv_len, int* queue, int* error_word, void* scratch, long long scratch_bytes, int* counters, int counters_len,
+    cudaStream_t stream) {
+  if (tiles == 0) return MLR_OK;
+  if (tiles < 0 || q_rows <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || page_size <= 0 || window < 0 ||
+      chunk < 0 || softcap < 0.f || q_stride < (long long)heads * head_dim || table_width <= 0 || pool_pages <= 0 ||
+      queue == nullptr || error_word == nullptr)
+    return MLR_BAD_SIZE;
+  if (head_dim != 64 && head_dim != 128) return MLR_BAD_SIZE;
+  if ((long long)tiles * heads >= (1ll << 30)) return MLR_TOO_LARGE;
+  const int page_shift = fa_shift_of(page_size);
+  if (page_shift < 3) return MLR_BAD_SIZE;
+  if (((uintptr_t)pool & 15) || ((uintptr_t)q & 15) || q_stride % 8 || ((uintptr_t)gate & 3) || gate_stride % 2)
+    return MLR_BAD_ALIGNMENT;
+  const long long pool_rows = (long long)pool_pages * kv_heads * page_size;
+  if (pool_rows >= (1ll << 31)) return MLR_TOO_LARGE;
+  const float log2e = 1.4426950408889634f;
+  FaScore score;
+  score.capped = softcap > 0.f;
+  score.in_scale = score.capped ? scale / softcap : scale * log2e;
+  score.out_scale = score.capped ? softcap * log2e : 1.f;
+  score.chunk = chunk;
+  score.slopes = slopes;
+  score.sinks = sinks;
+  score.gate = (const bf16*)gate;
+  score.gate_stride = gate_stride;
+  if (head_dim == 64)
+    return fa_launch<64, true>(q, pool, pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot,
+                               table_width, tiles, q_rows, heads, kv_heads, page_size, page_shift, pool_rows, window, scale,
+                               max_kv_len, queue, error_word, scratch, scratch_bytes, counters, counters_len, stream, q_stride,
+                               score);
+  return fa_launch<128, true>(q, pool, pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot,
+                              table_width, tiles, q_rows, heads, kv_heads, page_size, page_shift, pool_rows, window, scale,
+                              max_kv_len, queue, error_word, scratch, scratch_bytes, counters, counters_len, stream, q_stride,
+                              score);
 }

@@ -1664,7 +1664,23 @@ class CudaOps:
                 counters = self._workspace(q.device)["attention_counters"]
             launch(True, key if fused_store else None, (_ptr(None if only_decode else batch.plan["decode_seg"]), _ptr(None)),
                    batch.num_decode, partial, counters, splits, "shaped attention (decode)")
-        if batch.counts["wide"] > 0:
+        if (batch.counts["big"] > 0 and self.use_tcgen05_attention and dim in (64, 128) and page_size >= 8
+                and page_size & (page_size - 1) == 0 and q.storage_offset() % q.stride(0) == 0):
+            # prompt portions with the scores and P V on tcgen05
+            space = self._workspace(q.device)
+            longest = int(batch.max_kv_len)
+            if chunk or window:
+                # no item of 128 rows sees more keys than its rows' reach
+                longest = min(longest, min(int(chunk) or 1 << 30, int(window) or 1 << 30) + 128)
+            _check(build.load_library("attention_tcgen05").mlr_attention_shaped_prefill_tcgen05(
+                *q_view, _ptr(k_pool), _ptr(out), _ptr(batch.plan["big_tile_seg"]), _ptr(batch.plan["big_tile_row0"]),
+                *segments, batch.counts["big"], rows, heads, kv_heads, dim, page_size, k_pool.shape[0], int(window), int(chunk),
+                ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(slopes), _ptr(sink), *gate_view, longest,
+                _ptr(space["prefill_queue"]), _ptr(space["error_word"]),
+                _ptr(space["prefill_scratch"] if self.split_prefill_items else None),
+                ctypes.c_longlong(space["prefill_scratch"].numel()), _ptr(space["prefill_counters"]),
+                space["prefill_counters"].numel(), _stream()), "shaped attention (prefill, tcgen05)")
+        elif batch.counts["wide"] > 0:
             launch(False, None, (_ptr(batch.plan["wide_tile_seg"]), _ptr(batch.plan["wide_tile_row0"])),
                    batch.counts["wide"], None, None, 1, "shaped attention (prefill)")
         return out
