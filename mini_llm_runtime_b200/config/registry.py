@@ -20,6 +20,7 @@ from .rozesun import RozesunConfig, rozesun_model_spec
 from .spec import ModelSpec
 from .vetevik import VetevikConfig, vetevik_model_spec
 from .zazasun import ZazasunConfig, zazasun_model_spec
+from .zugarax import ZugaraxConfig, zugarax_model_spec
 
 
 @dataclass(frozen=True)
@@ -89,3 +90,4 @@ register_architecture(RozesunConfig.architecture, RozesunConfig.from_dict, rozes
 register_architecture(BopilornConfig.architecture, BopilornConfig.from_dict, bopilorn_model_spec)
 register_architecture(RatilornConfig.architecture, RatilornConfig.from_dict, ratilorn_model_spec)
 register_architecture(VetevikConfig.architecture, VetevikConfig.from_dict, vetevik_model_spec)
+register_architecture(ZugaraxConfig.architecture, ZugaraxConfig.from_dict, zugarax_model_spec)

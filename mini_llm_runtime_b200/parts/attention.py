@@ -404,19 +404,23 @@ class HeadNormAttention(PagedAttention):
 
 
 class ShapedAttention(PagedAttention):
-    """Grouped-query causal softmax attention without a rotation, whose scores are bent and limited by optional
-    pieces that other designs can combine.
+    """Grouped-query causal softmax attention whose queries, keys and scores are shaped by optional pieces that
+    other designs can combine.
 
     q = Wq x [heads * dim], k = Wk x [kv_heads * dim], v = Wv x [kv_heads * vdim], no biases;
-    ``keys_are_values``: v = k as projected, there is no Wv and only keys are cached.  Query head h reads
-    key/value head h // (heads / kv_heads).  score = (q . k) * ``scale``; ``softcap`` c > 0: score <- c tanh(score /
+    ``keys_are_values``: v = k as projected, there is no Wv and only keys are cached.  ``qk_norm``: every q and k
+    head is divided by its root mean square over dim (``eps`` inside the root) and multiplied by a learned weight
+    [dim] shared by the heads (``q.norm``, ``k.norm``).  ``rope_base``: then the first ``rope_dims`` entries of
+    every q and k head are turned by the position (``rope_layout``, ``rope_scaling``: see ``PairedRope``).  Query
+    head h reads key/value head h // (heads / kv_heads).  score = (q . k) * ``scale``; ``softcap`` c > 0: score <- c tanh(score /
     c); ``slopes`` (a number per head): slope_h * (i - j) off the score; ``chunk`` n > 0: position i sees only
     its own chunk of n positions (counted from the request's start), ``window`` n > 0: only its last n; ``sink``:
-    exp(sink_h), a learned number per head, joins the softmax's denominator; ``gate``: the concatenated heads are
+    exp(sink_h) joins the softmax's denominator, sink_h a learned number per head (``learned`` or True) or zero
+    for every head (``zero``: one is added to the denominator); ``gate``: the concatenated heads are
     multiplied by sigmoid(Wg x) before Wo.
 
-    32-bit: scores, cap, bias, softmax and the sums over keys.  In bfloat16 the projections, the cached keys and
-    values, the gate's projection and the attention's output are bfloat16."""
+    32-bit: norms, angles and rotation, scores, cap, bias, softmax and the sums over keys.  In bfloat16 the
+    projections, the cached keys and values, the gate's projection and the attention's output are bfloat16."""
 
     def __init__(self, spec, compute_dtype):
         super().__init__(spec, compute_dtype)
@@ -431,16 +435,32 @@ class ShapedAttention(PagedAttention):
         self.softcap = float(a.get("softcap") or 0.0)
         self.chunk = int(a.get("chunk") or 0)
         self.window = int(a.get("window") or 0)
-        self.has_sink = bool(a.get("sink", False))
+        sink = a.get("sink", False)
+        self.sink_kind = "learned" if sink is True else str(sink or "none")
+        if self.sink_kind not in ("none", "learned", "zero"):
+            raise ValueError(f"unknown sink {sink!r}; known: none, learned, zero")
         self.has_gate = bool(a.get("gate", False))
+        self.qk_norm = bool(a.get("qk_norm", False))
+        self.eps = float(a.get("eps", 0.0))
+        self.position = None
+        if a.get("rope_base"):
+            rope_dims = int(a.get("rope_dims", self.dim))
+            if rope_dims % 2 or not 0 < rope_dims <= self.dim:
+                raise ValueError("the rotation covers an even number of entries, at most dim")
+            self.position = build_part("position", PartSpec("rope_pairs", {
+                "head_dim": rope_dims, "theta": float(a["rope_base"]), "layout": a.get("rope_layout", "half"),
+                "scaling": dict(a.get("rope_scaling") or {})}), compute_dtype)
+        self.prepared = self.qk_norm or self.position is not None      # q and k pass a kernel before the attention
         self.slope_values = a.get("slopes")
         if self.heads % self.kv_heads:
             raise ValueError("heads must be divisible by kv_heads")
         if self.keys_are_values and self.vdim != self.dim:
             raise ValueError("keys that are values have one size")
+        if self.keys_are_values and self.prepared:
+            raise ValueError("keys that are values are used as projected")
         if self.slope_values is not None and len(self.slope_values) != self.heads:
             raise ValueError("one distance slope per head")
-        self.w_in = self.w_o = self.sink = self.slopes = None
+        self.w_in = self.w_o = self.sink = self.slopes = self.q_norm = self.k_norm = None
 
     def cache_need(self):
         value_dim = 0 if self.keys_are_values else (None if self.vdim == self.dim else self.vdim)
@@ -458,16 +478,29 @@ class ShapedAttention(PagedAttention):
         p, h = self.prefix, self.hidden_size
         out = {p + name: TensorSpec((rows, h)) for name, rows in self._sizes().items()}
         out[p + "o"] = TensorSpec((h, self.heads * self.vdim))
-        if self.has_sink:
+        if self.sink_kind == "learned":
             out[p + "sink"] = TensorSpec((self.heads,), init="bias")
+        if self.qk_norm:
+            out[p + "q.norm"] = TensorSpec((self.dim,), init="norm")
+            out[p + "k.norm"] = TensorSpec((self.dim,), init="norm")
         return out
 
     def load(self, tensors, device):
         p = self.prefix
+
+        def f32(name):
+            return tensors[p + name].to(device=device, dtype=torch.float32).contiguous()
+
         self.w_in = self._to_compute(torch.cat([tensors[p + name] for name in self._sizes()], dim=0), device)
         self.w_o = self._to_compute(tensors[p + "o"], device)
-        if self.has_sink:
-            self.sink = tensors[p + "sink"].to(device=device, dtype=torch.float32).contiguous()
+        if self.sink_kind == "learned":
+            self.sink = f32("sink")
+        elif self.sink_kind == "zero":
+            self.sink = torch.zeros(self.heads, dtype=torch.float32, device=device)
+        if self.qk_norm:
+            self.q_norm, self.k_norm = f32("q.norm"), f32("k.norm")
+        if self.position is not None:
+            self.position.load({}, device)
         if self.slope_values is not None:
             self.slopes = torch.tensor(self.slope_values, dtype=torch.float32, device=device)
 
@@ -478,10 +511,18 @@ class ShapedAttention(PagedAttention):
         for name, width in self._sizes().items():
             parts[name] = projected[:, at:at + width]
             at += width
-        mixed = k.shaped_attention(parts["q"], parts["k"], parts.get("v"), view.slots, view.k_pool, view.v_pool,
+        q, key, value = parts["q"], parts["k"], parts.get("v")
+        if self.prepared:
+            q = k.head_prepare(q, key, value, ctx.positions, self.q_norm, self.k_norm, self.eps,
+                               None if self.position is None else self.position.rotary_frequencies(),
+                               1.0 if self.position is None else self.position.magnitude,
+                               self.position is not None and self.position.interleaved, view.slots, view.k_pool, view.v_pool,
+                               self.heads, self.kv_heads, self.dim, self.vdim, writes_cache)
+            key = value = None         # in the pages already
+        mixed = k.shaped_attention(q, key, value, view.slots, view.k_pool, None if self.keys_are_values else view.v_pool,
                                    self._batch(ctx, view), self.heads, self.kv_heads, self.dim, self.vdim, self.scale,
                                    softcap=self.softcap, slopes=self.slopes, window=self.window, chunk=self.chunk,
-                                   sink=self.sink, gate=parts.get("g"), write_kv=writes_cache)
+                                   sink=self.sink, gate=parts.get("g"), write_kv=writes_cache and not self.prepared)
         return k.linear(mixed, self.w_o, out_dtype=torch.float32)
 
 

@@ -19,13 +19,17 @@ class PreNormResidual(Block):
     time.  Steps of few rows (decode) then run without norm kernels: the products apply the row
     scale themselves and the products that end the mixer and the feed-forward add their result
     into the stream in place.  Steps of many rows keep the arrangement below, with norm kernels
-    that only scale.  The float32 path keeps the reference's order of operations."""
+    that only scale.  The float32 path keeps the reference's order of operations.
+
+    The stream's dtype is the embedding's: with norms that read a 32-bit stream (``StreamRMSNorm``) and sublayers
+    that hand back 32-bit rows the same arrangement sums in 32-bit.  A layer without a feed-forward ends after
+    the mixer."""
 
     folded = False
 
     def finish_load(self, compute_dtype):
         if (compute_dtype == torch.bfloat16 and self.mixer.supports_norm_fusion
-                and self.feed_forward.supports_norm_fusion):
+                and self.feed_forward is not None and self.feed_forward.supports_norm_fusion):
             first, second = self.mixer_norm.fold(), self.feed_forward_norm.fold()
             if first is None or second is None:
                 raise ValueError("a norm that cannot be folded must say so before it is asked to")
@@ -46,6 +50,8 @@ class PreNormResidual(Block):
         else:
             normed = self.mixer_norm.add_forward(residual, pending)
         mixed = self.mixer.forward(normed, ctx, view, writes_cache)
+        if self.feed_forward is None:
+            return residual, mixed
         normed = self.feed_forward_norm.add_forward(residual, mixed)
         return residual, self.feed_forward.forward(normed, ctx)
 

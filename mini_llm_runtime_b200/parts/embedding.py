@@ -80,7 +80,7 @@ class TiedHead(Head):
 
 class LinearHead(Head):
     """logits = x H^T with the head's own matrix: ``<prefix>weight``, or the checkpoint name the
-    spec gives as ``tensor``."""
+    spec gives as ``tensor``.  ``softcap`` c > 0: logits <- c tanh(logits / c) (in 32-bit)."""
 
     graph_safe = True
 
@@ -89,6 +89,7 @@ class LinearHead(Head):
         self.vocab_size = int(self.args["vocab_size"])
         self.hidden_size = int(self.args["hidden_size"])
         self.tensor = self.args.get("tensor") or self.prefix + "weight"
+        self.softcap = float(self.args.get("softcap") or 0.0)
         self.weight: torch.Tensor | None = None
 
     def tensors(self):
@@ -98,7 +99,8 @@ class LinearHead(Head):
         self.weight = self._to_compute(tensors[self.tensor], device)
 
     def forward(self, x, embedding):
-        return ops.current().linear(x, self.weight, None, out_dtype=torch.float32)
+        logits = ops.current().linear(x, self.weight, None, out_dtype=torch.float32)
+        return ops.current().softcap_(logits, self.softcap) if self.softcap > 0 else logits
 
 
 class TokenPositionEmbedding(Embedding):

@@ -63,7 +63,8 @@ class GatedMLP(FeedForward):
     down(g * sigmoid(slope * g) * (u + 1)) where g = min(gate(x), limit) and u = clamp(up(x), -limit,
     limit) (``limit`` from the spec, ``slope`` 1.702 unless given).  The result leaves in 32-bit floats, for
     arrangements that sum into a 32-bit stream.  ``names`` gives the three checkpoint names after
-    the prefix.  gate and up are stacked like SwiGLU's."""
+    the prefix.  gate and up are stacked like SwiGLU's.  ``bias`` (clamped gate only): every product has a bias,
+    its checkpoint name that of the matrix + ".b"."""
 
     graph_safe = True
 
@@ -79,14 +80,20 @@ class GatedMLP(FeedForward):
         if self.activation == "clamped_swish" and not self.limit > 0:
             raise ValueError("the clamped gate needs a positive limit")
         self.names = tuple(self.args.get("names") or ("gate_proj.weight", "up_proj.weight", "down_proj.weight"))
-        self.w_gate_up = self.w_down = None
+        self.bias = bool(self.args.get("bias", False))
+        if self.bias and self.activation != "clamped_swish":
+            raise ValueError("biases are known for the clamped gate only")
+        self.w_gate_up = self.w_down = self.b_gate_up = self.b_down = None
         self.block = self.intermediate_size
 
     def tensors(self):
         gate, up, down = (self.prefix + name for name in self.names)
-        return {gate: TensorSpec((self.intermediate_size, self.hidden_size)),
-                up: TensorSpec((self.intermediate_size, self.hidden_size)),
-                down: TensorSpec((self.hidden_size, self.intermediate_size))}
+        out = {gate: TensorSpec((self.intermediate_size, self.hidden_size)),
+               up: TensorSpec((self.intermediate_size, self.hidden_size)),
+               down: TensorSpec((self.hidden_size, self.intermediate_size))}
+        if self.bias:
+            out.update({name + ".b": TensorSpec(spec.shape[:1], init="bias") for name, spec in list(out.items())})
+        return out
 
     def load(self, tensors, device):
         gate, up, down = (tensors[self.prefix + name] for name in self.names)
@@ -98,14 +105,19 @@ class GatedMLP(FeedForward):
             stacked = torch.cat([gate, up], dim=0)
         self.w_gate_up = self._to_compute(stacked, device)
         self.w_down = self._to_compute(down, device)
+        if self.bias:
+            gate_b, up_b, down_b = (tensors[self.prefix + name + ".b"] for name in self.names)
+            stacked = torch.cat([gate_b.view(-1, self.block), up_b.view(-1, self.block)], dim=1).reshape(-1)
+            self.b_gate_up = self._to_compute(stacked, device)
+            self.b_down = self._to_compute(down_b, device)
 
     def forward(self, x, ctx):
         k = ops.current()
         if self.activation == "clamped_swish":
-            hidden = k.linear_clamped_gate(x, self.w_gate_up, self.block, self.limit, self.slope)
+            hidden = k.linear_clamped_gate(x, self.w_gate_up, self.block, self.limit, self.slope, bias=self.b_gate_up)
         else:
             hidden = k.linear_gated(x, self.w_gate_up, self.block, self.activation)
-        return k.linear(hidden, self.w_down, out_dtype=torch.float32)
+        return k.linear(hidden, self.w_down, self.b_down, out_dtype=torch.float32)
 
 
 register_part("feed_forward", "swiglu", SwiGLU)

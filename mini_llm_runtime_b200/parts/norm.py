@@ -181,8 +181,10 @@ class StreamRMSNorm(Norm):
 
     def add_forward(self, residual, delta, post=None, offset=None):
         if post is None:
-            ops.current().add_residual(residual, delta)
-            return self.forward(residual, offset)
+            if offset is not None:
+                ops.current().add_residual(residual, delta)
+                return self.forward(residual, offset)
+            return self.forward(residual, delta)      # rows added and normalised in one pass
         if post.eps != self.eps or getattr(post, "groups", 1) != self.groups:
             post.add_into(residual, delta)
             return self.forward(residual, offset)

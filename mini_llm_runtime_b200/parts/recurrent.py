@@ -12,6 +12,8 @@ recurrence; the mixer's output projection leaves 32-bit rows for a 32-bit residu
            out = Wo (o / rms(o) * norm * silu(Wg x_g)).
 ``state_space``  a selective state-space layer with a scalar decay per head (Mamba-2, "state-space
            duality"), see ``StateSpaceMixer``.
+``matrix_memory``  a memory written with exponential gates and read through a normaliser, see
+           ``MatrixMemoryMixer``.
 ``gated_delta_rule``  a delta rule with a scalar decay and step size per head, see ``DeltaRuleMixer``.
 ``hgrn2``  gated linear attention whose forget gate also sets what is written:
            f_t = l + (1 - l) sigmoid(Wf x + b);  S <- diag(f_t) S + (1 - f_t) v_t^T;
@@ -285,7 +287,79 @@ class DeltaRuleMixer(Mixer):
         return k.linear(gated, self.w_o, out_dtype=torch.float32)
 
 
+class MatrixMemoryMixer(Mixer):
+    """Matrix memory with exponential gates (the mLSTM of xLSTM).
+
+    q = Wq x * dim^-0.5 and k = Wk x [heads * dim], v = Wv x [heads * vdim].  Per head and token a logarithm of the
+    input gate i = cap tanh((Wi x + bi) / cap) and one of the forget gate f = logsigmoid(cap tanh((Wf x + bf) /
+    cap)), cap = ``gate_cap``.  The memory S [dim, vdim] and its normaliser n [dim] are kept relative to the
+    exponential of a running maximum m, so that no gate overflows:  m_t = max(f + m_{t-1}, i),  S_t = e^(f + m_{t-1} -
+    m_t) S_{t-1} + e^(i - m_t) k v^T,  n_t likewise with k alone,  o = S_t^T q / (max(|n_t . q|, e^(-m_t)) +
+    ``guard``).  Every head's o is divided by its root mean square, the heads together are multiplied by ``norm``
+    [heads * vdim] and by sigmoid(Wg x); then Wo.
+
+    Per request the layer carries, in 32-bit, S with n behind it (kept transposed, n as one more value channel:
+    [heads, vdim + 1, dim]) and m; all start at zero.  Everything between the projections and Wo is 32-bit."""
+
+    graph_safe = True
+    NAMES = ("q", "k", "v", "g", "i", "f")
+
+    def __init__(self, spec, compute_dtype):
+        super().__init__(spec, compute_dtype)
+        a = self.args
+        self.hidden_size = int(a["hidden_size"])
+        self.heads = int(a["heads"])
+        self.dim = int(a["dim"])
+        self.vdim = int(a["vdim"])
+        self.eps = float(a["eps"])
+        self.gate_cap = float(a["gate_cap"])
+        self.guard = float(a.get("guard", 1e-6))
+        self.qk, self.inner = self.heads * self.dim, self.heads * self.vdim
+        self.w_in = self.w_o = self.input_bias = self.forget_bias = self.norm = None
+
+    def cache_need(self):
+        return (StateNeed((self.heads, self.vdim + 1, self.dim), torch.float32, "state"),
+                StateNeed((self.heads,), torch.float32, "maximum"))
+
+    def _sizes(self):
+        return dict(zip(self.NAMES, (self.qk, self.qk, self.inner, self.inner, self.heads, self.heads)))
+
+    def tensors(self):
+        p, h = self.prefix, self.hidden_size
+        out = {p + name: TensorSpec((rows, h)) for name, rows in self._sizes().items()}
+        out.update({p + "i.b": TensorSpec((self.heads,), init="bias"), p + "f.b": TensorSpec((self.heads,), init="bias"),
+                    p + "norm": TensorSpec((self.inner,), init="norm"), p + "o": TensorSpec((h, self.inner))})
+        return out
+
+    def load(self, tensors, device):
+        p = self.prefix
+        # one product yields [q | k | v | g | i | f], filled up with zeros so that its rows start at 16-byte boundaries
+        rows = [tensors[p + name] for name in self.NAMES]
+        fill = -sum(part.shape[0] for part in rows) % 8
+        if fill:
+            rows.append(torch.zeros((fill, self.hidden_size), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = self._to_compute(torch.cat(rows, dim=0), device)
+        self.w_o = self._to_compute(tensors[p + "o"], device)
+        self.input_bias = _float(tensors[p + "i.b"], device)
+        self.forget_bias = _float(tensors[p + "f.b"], device)
+        self.norm = _float(tensors[p + "norm"], device)
+
+    def forward(self, x, ctx, view, writes_cache):
+        k = ops.current()
+        projected = k.linear(x, self.w_in, out_dtype=torch.float32)
+        parts, at = {}, 0
+        for name, width in self._sizes().items():
+            parts[name] = projected[:, at:at + width]
+            at += width
+        mixed = k.matrix_memory(parts["q"], parts["k"], parts["v"], parts["i"], parts["f"], self.input_bias,
+                                self.forget_bias, self.gate_cap, self.guard, parts["g"], self.norm, self.eps,
+                                view.states["state"], view.states["maximum"], ctx, self.heads, self.dim, self.vdim,
+                                self.compute_dtype)
+        return k.linear(mixed, self.w_o, out_dtype=torch.float32)
+
+
 register_part("mixer", "wkv", WKVMixer)
+register_part("mixer", "matrix_memory", MatrixMemoryMixer)
 register_part("mixer", "gated_delta_rule", DeltaRuleMixer)
 register_part("mixer", "state_space", StateSpaceMixer)
 register_part("mixer", "hgrn2", HGRN2Mixer)

@@ -53,22 +53,35 @@ class PairedRope(RotateHalfRope):
     ``layout="interleaved"``, (2i, 2i + 1); it turns by position * theta^(-2i/head_dim).  The frequencies
     are evaluated in 64-bit and rounded once.
 
-    ``scaling`` = {factor, original, fast, slow} stretches the long wavelengths for contexts beyond the
-    ``original`` one: with pair(t) = head_dim * ln(original / (2 pi t)) / (2 ln theta) the index of the
+    ``scaling`` stretches the long wavelengths for contexts beyond the ``original`` one.  Its ``kind`` is
+    ``ramp`` (if none is given) or ``bands``.
+
+    ``ramp``, {factor, original, fast, slow}: with pair(t) = head_dim * ln(original / (2 pi t)) / (2 ln theta) the index of the
     pair that makes t turns over the original context, low = max(floor(pair(fast)), 0), high =
     min(ceil(pair(slow)), head_dim - 1) and ramp_i = clamp((i - low) / max(high - low, 0.001), 0, 1), pair
     i gets f_i / factor * ramp_i + f_i * (1 - ramp_i); ``magnitude`` = 0.1 ln(factor) + 1 multiplies
-    sine and cosine (1 without scaling)."""
+    sine and cosine (1 without this scaling).
+
+    ``bands``, {factor, original, low, high}: with n_i = original * f_i / (2 pi), the turns pair i makes over the
+    original context, f_i stays where n_i > high, becomes f_i / factor where n_i < low, and in between is
+    blended, (1 - s) f_i / factor + s f_i with s = (n_i - low) / (high - low)."""
+
+    SCALINGS = {"ramp": ("factor", "original", "fast", "slow"), "bands": ("factor", "original", "low", "high")}
 
     def __init__(self, spec, compute_dtype):
         layout = str(spec.args.get("layout", "half"))
         if layout not in ("half", "interleaved"):
             raise ValueError(f"unknown pair layout {layout!r}; known: half, interleaved")
         scaling = dict(spec.args.get("scaling") or {})
-        if scaling and any(name not in scaling for name in ("factor", "original", "fast", "slow")):
-            raise ValueError("a frequency scaling needs factor, original, fast and slow")
+        self.scaling_kind = str(scaling.pop("kind", "ramp"))
+        if self.scaling_kind not in self.SCALINGS:
+            raise ValueError(f"unknown frequency scaling {self.scaling_kind!r}; known: {', '.join(self.SCALINGS)}")
+        names = self.SCALINGS[self.scaling_kind]
+        if scaling and any(name not in scaling for name in names):
+            raise ValueError(f"a frequency scaling of this kind needs {', '.join(names)}")
         self.scaling = scaling
-        self.magnitude = 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling else 1.0
+        ramped = scaling and self.scaling_kind == "ramp"
+        self.magnitude = 0.1 * math.log(float(scaling["factor"])) + 1.0 if ramped else 1.0
         super().__init__(spec, compute_dtype)
         self.interleaved = layout == "interleaved"
 
@@ -79,6 +92,13 @@ class PairedRope(RotateHalfRope):
         if not self.scaling:
             return plain.to(torch.float32)
         factor, original = float(self.scaling["factor"]), float(self.scaling["original"])
+        if self.scaling_kind == "bands":
+            low, high = float(self.scaling["low"]), float(self.scaling["high"])
+            turns = original * plain / (2.0 * math.pi)
+            share = (turns - low) / (high - low) if high != low else torch.zeros_like(turns)
+            blended = (1.0 - share) * plain / factor + share * plain
+            scaled = torch.where(turns < low, plain / factor, torch.where(turns > high, plain, blended))
+            return scaled.to(torch.float32)
 
         def pair_of(turns: float) -> float:
             return n * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))

@@ -321,21 +321,25 @@ class FakeOps:
         gate, up = gate.clamp(max=limit), up.clamp(-limit, limit)
         return (gate * torch.sigmoid(slope * gate) * (up + 1.0)).to(gate_up.dtype)
 
-    def linear_clamped_gate(self, x, weight, block, limit, slope):
-        return self.clamped_gate(self.linear(x, weight), block, limit, slope)
+    def linear_clamped_gate(self, x, weight, block, limit, slope, bias=None):
+        return self.clamped_gate(self.linear(x, weight, bias), block, limit, slope)
+
+    def softcap_(self, x, cap):
+        return x.copy_(cap * torch.tanh(x / cap))
 
     def scale_(self, x, factor):
         x *= factor
         return x
 
     @staticmethod
-    def _turn(vector, positions, frequencies, interleaved):
-        """vector [rows, ..., n]: the first 2 * len(frequencies) entries turned by the rows' positions."""
+    def _turn(vector, positions, frequencies, interleaved, magnitude=1.0):
+        """vector [rows, ..., n]: the first 2 * len(frequencies) entries turned by the rows' positions, sine and
+        cosine times ``magnitude``."""
         pairs = frequencies.shape[0]
         out = vector.clone()
         angle = positions.float()[:, None] * frequencies[None, :]
         shape = (vector.shape[0],) + (1,) * (vector.dim() - 2) + (pairs,)
-        cos, sin = torch.cos(angle).view(shape), torch.sin(angle).view(shape)
+        cos, sin = torch.cos(angle).view(shape) * magnitude, torch.sin(angle).view(shape) * magnitude
         first = torch.arange(pairs) * 2 if interleaved else torch.arange(pairs)
         second = first + 1 if interleaved else first + pairs
         u, v = vector[..., first], vector[..., second]
@@ -344,30 +348,31 @@ class FakeOps:
         return out
 
     def latent_prepare(self, down, q_at, q_rank, c_at, rank, rot, q_weight, c_weight, eps, positions, frequencies,
-                       interleaved, slots, pool, write=True):
+                       interleaved, slots, pool, write=True, magnitude=1.0):
         def normed(t, weight):
             return t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps) * weight
 
-        q_latent = normed(down[:, q_at:q_at + q_rank], q_weight).to(pool.dtype)
+        q_latent = normed(down[:, q_at:q_at + q_rank], q_weight).to(pool.dtype) if q_rank else None
         if write:
             latent = normed(down[:, c_at:c_at + rank], c_weight)
-            turned = self._turn(down[:, c_at + rank:c_at + rank + rot], positions, frequencies, interleaved)
+            turned = self._turn(down[:, c_at + rank:c_at + rank + rot], positions, frequencies, interleaved, magnitude)
             rows, page_size = torch.cat([latent, turned], dim=1).to(pool.dtype), pool.shape[2]
             for t in range(down.shape[0]):
                 page, offset = divmod(int(slots[t]), page_size)
                 pool[page, 0, offset, :] = rows[t]
         return q_latent
 
-    def absorb_queries(self, q, weight, heads, dim, rot, rank, positions, frequencies, interleaved):
-        q = q.view(-1, heads, dim + rot)
+    def absorb_queries(self, q, weight, heads, dim, rot, rank, positions, frequencies, interleaved, magnitude=1.0):
+        q = q.reshape(-1, heads, dim + rot)
         plain = torch.einsum("rhd,hdc->rhc", q[..., :dim], weight.float().view(heads, dim, rank))
-        turned = self._turn(q[..., dim:], positions, frequencies, interleaved)
+        turned = self._turn(q[..., dim:], positions, frequencies, interleaved, magnitude)
         return torch.cat([plain, turned], dim=-1).reshape(q.shape[0], -1).to(weight.dtype)
 
     def latent_values(self, mixed, weight, heads, vdim, rank, gate, gate_per_head):
         out = torch.einsum("rhc,hvc->rhv", mixed.view(-1, heads, rank), weight.float().view(heads, vdim, rank))
-        gate = torch.sigmoid(gate.float())
-        out = out * (gate[:, :, None] if gate_per_head else gate.view(-1, heads, vdim))
+        if gate is not None:
+            gate = torch.sigmoid(gate.float())
+            out = out * (gate[:, :, None] if gate_per_head else gate.view(-1, heads, vdim))
         return out.reshape(mixed.shape[0], -1).to(weight.dtype)
 
     def latent_attention(self, q, pool, batch, heads, rank, rot, scale, window, sink):
@@ -561,7 +566,7 @@ class FakeOps:
                     if slot >= 0:
                         page, offset = divmod(slot, page_size)
                         pool[page, :, offset, :] = source[t].reshape(kv_heads, -1)
-        if value is None:
+        if v_pool is None:
             v_pool = k_pool
         out = torch.empty((rows, heads * vdim), dtype=q.dtype)
         q3 = q.float().reshape(rows, heads, dim)
@@ -590,6 +595,46 @@ class FakeOps:
                     mixed = mixed * torch.sigmoid(gate[start + r].float())
                 out[start + r] = mixed.to(q.dtype)
         return out
+
+    def head_prepare(self, q, key, value, positions, q_weight, k_weight, eps, freq, magnitude, interleaved, slots, k_pool,
+                     v_pool, heads, kv_heads, dim, vdim, write_kv=True):
+        def prepared(x, count, weight):
+            x = x.float().reshape(-1, count, dim)
+            if weight is not None:
+                x = self._rms(x, eps) * weight
+            if freq is not None:
+                x = self._turn(x, positions, freq, interleaved, magnitude)
+            return x.to(k_pool.dtype)
+
+        if write_kv:
+            keys, values = prepared(key, kv_heads, k_weight), value.reshape(-1, kv_heads, vdim)
+            for t in range(q.shape[0]):
+                slot = int(slots[t])
+                if slot >= 0:
+                    page, offset = divmod(slot, k_pool.shape[2])
+                    k_pool[page, :, offset, :] = keys[t]
+                    v_pool[page, :, offset, :] = values[t]
+        return prepared(q, heads, q_weight).reshape(q.shape[0], -1)
+
+    # ---- matrix memory with exponential gates
+    def matrix_memory(self, q, k, v, i_raw, f_raw, i_bias, f_bias, cap, guard, gate, weight, eps, state, maximum, ctx, heads,
+                      dim, vdim, out_dtype):
+        log_in = cap * torch.tanh((i_raw + i_bias) / cap)
+        log_forget = torch.nn.functional.logsigmoid(cap * torch.tanh((f_raw + f_bias) / cap))
+        out = torch.empty((q.shape[0], heads, vdim), dtype=torch.float32)
+        for segment in ctx.segments:
+            S, m = state[segment.slot], maximum[segment.slot]                   # [heads, vdim + 1, dim], [heads]
+            for row in range(segment.row_start, segment.row_start + segment.length):
+                new = torch.maximum(log_forget[row] + m, log_in[row])
+                keep, write = torch.exp(log_forget[row] + m - new), torch.exp(log_in[row] - new)
+                m = new
+                values = torch.cat([v[row].view(heads, vdim), torch.ones(heads, 1)], dim=1) * write[:, None]
+                S = keep[:, None, None] * S + values[:, :, None] * k[row].view(heads, 1, dim)
+                read = torch.einsum("hvd,hd->hv", S, q[row].view(heads, dim) * dim ** -0.5)
+                out[row] = read[:, :vdim] / (torch.maximum(read[:, vdim:].abs(), torch.exp(-m)[:, None]) + guard)
+            state[segment.slot], maximum[segment.slot] = S, m
+        normed = self._rms(out, eps).reshape(q.shape[0], -1)
+        return (normed * weight * torch.sigmoid(gate)).to(out_dtype)
 
     def delta_rule_scan(self, q, k, v, a, b, dt_bias, A_log, state, ctx, heads, kv_heads, dim, vdim, unit_eps):
         def unit(x):
