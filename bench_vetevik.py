@@ -141,7 +141,7 @@ def kernel_points(size, peak):
         row_bytes = rows * heads * dim * 2
         slopes, sink = torch.rand(heads, device="cuda") * 0.01, vector(heads)
         record(f"shaped_attention.{label}",
-               _time(lambda: k.shaped_attention(q, key, None, slots, k_pool, k_pool, batch, heads, kv_heads, dim, dim, dim ** -0.5,
+               _time(lambda: k.shaped_attention(q, key, None, slots, k_pool, None, batch, heads, kv_heads, dim, dim, dim ** -0.5,
                                                 softcap=SOFTCAP, slopes=slopes, chunk=s["chunk"], sink=sink, gate=gate), flush),
                key_bytes + 3 * row_bytes, pairs * heads * 4 * dim)
         q_plain = q.contiguous()

@@ -48,7 +48,8 @@ __global__ void __launch_bounds__(128)
 latent_prepare_kernel(const float* down, long long down_stride, int q_at, int q_rank, int c_at, int rank, int rot,
                       const float* __restrict__ q_weight, const float* __restrict__ c_weight,
                       const int* positions, const float* __restrict__ frequencies, int pairs, int interleaved,
-                      const long long* slots, T* __restrict__ q_latent, T* __restrict__ pool, float eps, int write) {
+                      const long long* slots, T* __restrict__ q_latent, T* __restrict__ pool, float eps, int write,
+                      float magnitude) {
   pdl_trigger();
   __shared__ float scratch[32];
   const int row = blockIdx.x;
@@ -67,7 +68,7 @@ latent_prepare_kernel(const float* down, long long down_stride, int q_at, int q_
   for (int d = threadIdx.x; d < q_rank; d += blockDim.x) sq_q = fmaf(in[q_at + d], in[q_at + d], sq_q);
   if (store)
     for (int d = threadIdx.x; d < rank; d += blockDim.x) sq_c = fmaf(in[c_at + d], in[c_at + d], sq_c);
-  {
+  if (q_rank > 0) {
     const float factor = 1.f / sqrtf(block_sum(sq_q, scratch) / (float)q_rank + eps);
     T* dst = q_latent + (size_t)row * q_rank;
     for (int d = threadIdx.x; d < q_rank; d += blockDim.x) dst[d] = from_float<T>(in[q_at + d] * factor * q_weight[d]);
@@ -82,6 +83,8 @@ latent_prepare_kernel(const float* down, long long down_stride, int q_at, int q_
     pair_places(i, pairs, interleaved, &a, &b);
     float sine, cosine, ya, yb;
     sincosf(position * frequencies[i], &sine, &cosine);
+    sine *= magnitude;
+    cosine *= magnitude;
     rotate_pair(r[a], r[b], sine, cosine, &ya, &yb);
     dst[rank + a] = from_float<T>(ya);
     dst[rank + b] = from_float<T>(yb);
@@ -95,14 +98,14 @@ latent_prepare_kernel(const float* down, long long down_stride, int q_at, int q_
 // (KN = 0) or [heads][K][N] (KN = 1), y in TO at y + r * y_row + h * y_head + n.  Sums run over k in
 // ascending order in float32.  Then, depending on `mode`:
 //   1  the `tail` numbers after x's K are copied behind y's N with their first 2 * pairs entries turned
-//      by the row's position (the turned part of an absorbed query);
+//      by the row's position, sine and cosine times `magnitude` (the turned part of an absorbed query);
 //   2  y is multiplied by sigmoid(g), g = gate[r * gate_row + (gate_per_head ? h : h * N + n)].
 struct HeadLinearArgs {
   const float* x; long long x_row; int x_head;
   long long y_row; int y_head;
   int rows, heads, N, K, kn, mode;
   int tail, pairs, interleaved;
-  const int* positions; const float* frequencies;
+  const int* positions; const float* frequencies; float magnitude;
   const float* gate; long long gate_row; int gate_per_head;
 };
 
@@ -190,6 +193,8 @@ head_linear_kernel(const T* __restrict__ w, TO* __restrict__ y, HeadLinearArgs p
         pair_places(i, p.pairs, p.interleaved, &a, &b);
         float sine, cosine, ya, yb;
         sincosf((float)p.positions[row] * p.frequencies[i], &sine, &cosine);
+        sine *= p.magnitude;
+        cosine *= p.magnitude;
         rotate_pair(src[a], src[b], sine, cosine, &ya, &yb);
         dst[d] = from_float<TO>(second ? yb : ya);
       }
@@ -556,18 +561,18 @@ MLR_DEFINE_PDL_SWITCH
 MLR_EXPORT int mlr_latent_prepare(const float* down, long long down_stride, int q_at, int q_rank, int c_at, int rank,
                                   int rot, const float* q_weight, const float* c_weight, const int* positions,
                                   const float* frequencies, int pairs, int interleaved, const long long* slots,
-                                  void* q_latent, void* pool, int rows, float eps, int write, int dtype,
+                                  void* q_latent, void* pool, int rows, float eps, float magnitude, int write, int dtype,
                                   cudaStream_t stream) {
   if (rows == 0) return MLR_OK;
-  if (rows < 0 || q_rank <= 0 || rank <= 0 || rot < 0 || pairs < 0 || 2 * pairs > rot) return MLR_BAD_SIZE;
+  if (rows < 0 || q_rank < 0 || rank <= 0 || rot < 0 || pairs < 0 || 2 * pairs > rot) return MLR_BAD_SIZE;
   if (dtype == MLR_F32)
     launch_kernel(latent_prepare_kernel<float>, dim3(rows), dim3(128), 0, stream, down, down_stride, q_at, q_rank, c_at,
                   rank, rot, q_weight, c_weight, positions, frequencies, pairs, interleaved, slots, (float*)q_latent,
-                  (float*)pool, eps, write);
+                  (float*)pool, eps, write, magnitude);
   else if (dtype == MLR_BF16)
     launch_kernel(latent_prepare_kernel<bf16>, dim3(rows), dim3(128), 0, stream, down, down_stride, q_at, q_rank, c_at,
                   rank, rot, q_weight, c_weight, positions, frequencies, pairs, interleaved, slots, (bf16*)q_latent,
-                  (bf16*)pool, eps, write);
+                  (bf16*)pool, eps, write, magnitude);
   else
     return MLR_BAD_DTYPE;
   return launch_status();
@@ -576,7 +581,7 @@ MLR_EXPORT int mlr_latent_prepare(const float* down, long long down_stride, int 
 // See HeadLinearArgs.  w_dtype: dtype of w; y_dtype: dtype of y.
 MLR_EXPORT int mlr_head_linear(const float* x, long long x_row, int x_head, const void* w, void* y, long long y_row,
                                int y_head, int rows, int heads, int N, int K, int kn, int mode, int tail, int pairs,
-                               int interleaved, const int* positions, const float* frequencies, const float* gate,
+                               int interleaved, const int* positions, const float* frequencies, float magnitude, const float* gate,
                                long long gate_row, int gate_per_head, int w_dtype, int y_dtype, cudaStream_t stream) {
   if (rows == 0) return MLR_OK;
   if (rows < 0 || heads <= 0 || N <= 0 || K <= 0 || tail < 0 || pairs < 0 || 2 * pairs > tail) return MLR_BAD_SIZE;
@@ -586,7 +591,7 @@ MLR_EXPORT int mlr_head_linear(const float* x, long long x_row, int x_head, cons
   HeadLinearArgs p;
   p.x = x; p.x_row = x_row; p.x_head = x_head; p.y_row = y_row; p.y_head = y_head; p.rows = rows; p.heads = heads;
   p.N = N; p.K = K; p.kn = kn; p.mode = mode; p.tail = mode == 1 ? tail : 0; p.pairs = pairs; p.interleaved = interleaved;
-  p.positions = positions; p.frequencies = frequencies; p.gate = gate; p.gate_row = gate_row; p.gate_per_head = gate_per_head;
+  p.positions = positions; p.frequencies = frequencies; p.magnitude = magnitude; p.gate = gate; p.gate_row = gate_row; p.gate_per_head = gate_per_head;
   const dim3 grid((N + HL_BN - 1) / HL_BN, (rows + HL_BM - 1) / HL_BM, heads);
   if (w_dtype == MLR_F32 && y_dtype == MLR_F32)
     launch_kernel(head_linear_kernel<float, float>, grid, dim3(128), 0, stream, (const float*)w, (float*)y, p);

@@ -333,7 +333,7 @@ struct HeadMmaArgs {
   long long y_row; int y_head;
   int rows, heads, N, K, kn, mode;
   int tail, pairs, interleaved;
-  const int* positions; const float* frequencies;
+  const int* positions; const float* frequencies; float magnitude;
   const float* gate; long long gate_row; int gate_per_head;
 };
 
@@ -465,6 +465,8 @@ head_linear_mma_kernel(const bf16* __restrict__ w, TO* __restrict__ y, HeadMmaAr
         const int a = p.interleaved ? 2 * i : i, b = p.interleaved ? 2 * i + 1 : i + p.pairs;
         float sine, cosine, ya, yb;
         sincosf((float)p.positions[row] * p.frequencies[i], &sine, &cosine);
+        sine *= p.magnitude;
+        cosine *= p.magnitude;
         rotate_pair(src[a], src[b], sine, cosine, &ya, &yb);
         dst[d] = from_float<TO>(second ? yb : ya);
       }
@@ -578,7 +580,7 @@ MLR_EXPORT int mlr_latent_attention_mma_decode(const void* q, const void* pool, 
 // takes the float32 kernel.
 MLR_EXPORT int mlr_head_linear_mma(const float* x, long long x_row, int x_head, const void* w, void* y, long long y_row,
                                    int y_head, int rows, int heads, int N, int K, int kn, int mode, int tail, int pairs,
-                                   int interleaved, const int* positions, const float* frequencies, const float* gate,
+                                   int interleaved, const int* positions, const float* frequencies, float magnitude, const float* gate,
                                    long long gate_row, int gate_per_head, int y_dtype, cudaStream_t stream) {
   if (rows == 0) return MLR_OK;
   if (rows < 0 || heads <= 0 || N <= 0 || K <= 0 || tail < 0 || pairs < 0 || 2 * pairs > tail) return MLR_BAD_SIZE;
@@ -590,7 +592,7 @@ MLR_EXPORT int mlr_head_linear_mma(const float* x, long long x_row, int x_head, 
   HeadMmaArgs p;
   p.x = x; p.x_row = x_row; p.x_head = x_head; p.y_row = y_row; p.y_head = y_head; p.rows = rows; p.heads = heads;
   p.N = N; p.K = K; p.kn = kn; p.mode = mode; p.tail = mode == 1 ? tail : 0; p.pairs = pairs; p.interleaved = interleaved;
-  p.positions = positions; p.frequencies = frequencies; p.gate = gate; p.gate_row = gate_row; p.gate_per_head = gate_per_head;
+  p.positions = positions; p.frequencies = frequencies; p.magnitude = magnitude; p.gate = gate; p.gate_row = gate_row; p.gate_per_head = gate_per_head;
   const bool few = rows <= 16;
   const dim3 grid((N + HM_COLS - 1) / HM_COLS, few ? 1 : (rows + 63) / 64, heads);
   if (y_dtype == MLR_BF16) {

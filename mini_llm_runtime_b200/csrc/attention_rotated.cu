@@ -12,6 +12,10 @@
 //                       Pairs are (i, i + n/2) or, interleaved, (2i, 2i + 1), n being the number of
 //                       turned entries.  All arithmetic is float32; sums have an order fixed by the
 //                       sizes, so a row's numbers do not depend on the rest of the batch.
+// mlr_head_prepare      the same place in front of another attention: every q and k head divided by its own root mean
+//                       square (times a weight shared by the heads; skipped without weights), then turned as above;
+//                       q goes out, k and the values as projected go into the cache pages.  Inputs are views of a
+//                       product in the compute dtype.
 // mlr_turn_heads        x[row, head, :n] turned in place by sign * position * freq[i] (the way back of
 //                       the values' rotation, applied to each head's attention output).
 #include "common.cuh"
@@ -344,6 +348,153 @@ rotated_prepare_kernel(const float* qkv, const int* positions, const float* __re
   }
 }
 
+struct HeadPrepareArgs {
+  const void *q, *k, *v;                       // rows of heads * dim, kv_heads * dim, kv_heads * vdim entries
+  long long q_stride, k_stride, v_stride;      // entries from row to row
+  const int* positions;
+  const float *q_weight, *k_weight;            // [dim] or null: no norm
+  const float* freq;                           // [rot / 2]
+  const long long* slots;
+  void *q_out, *k_pool, *v_pool;
+  int heads, kv_heads, dim, vdim, rot, interleaved, page_size, write_kv;
+  float eps, magnitude;
+};
+
+// One block per row.  PIECES > 0: heads in pieces of four entries, a group of `lanes` lanes per head (a power of
+// two), PIECES of them per lane, partners of the rotation in whole pieces; all of a lane's pieces and their partners
+// are asked for at once.  PIECES == 0: any sizes, a warp per head, entry by entry.
+template <typename T, int PIECES>
+__global__ void __launch_bounds__(256)
+head_prepare_kernel(const HeadPrepareArgs p, int lanes) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float tables[];      // rot / 2 sines, then rot / 2 cosines
+  const int r = blockIdx.x, half = p.rot / 2, D = p.dim;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  constexpr int WARPS = 256 / 32;
+  float* sine = tables;
+  float* cosine = tables + half;
+  const float position = (float)p.positions[r];
+  for (int i = threadIdx.x; i < half; i += 256) {
+    float s, c;
+    sincosf(position * p.freq[i], &s, &c);
+    sine[i] = s * p.magnitude;
+    cosine[i] = c * p.magnitude;
+  }
+  const long long slot = p.write_kv ? p.slots[r] : -1;
+  const bool store = slot >= 0;
+  const long long page = store ? slot / p.page_size : 0;
+  const int offset = store ? (int)(slot - page * p.page_size) : 0;
+  T* k_row = (T*)p.k_pool + ((size_t)page * p.kv_heads * p.page_size + offset) * D;      // head g: g * page_size * dim on
+  T* v_row = (T*)p.v_pool + ((size_t)page * p.kv_heads * p.page_size + offset) * p.vdim;
+  const T* q_in = (const T*)p.q + (size_t)r * p.q_stride;
+  const T* k_in = (const T*)p.k + (size_t)r * p.k_stride;
+  const T* v_in = (const T*)p.v + (size_t)r * p.v_stride;
+  T* q_out = (T*)p.q_out + (size_t)r * p.heads * D;
+  __syncthreads();
+  pdl_wait();
+  const int all_heads = p.heads + (store ? p.kv_heads : 0);
+
+  if (PIECES > 0) {
+    constexpr int N = PIECES > 0 ? PIECES : 1;
+    if (store)
+      for (int idx = threadIdx.x; idx < p.kv_heads * (p.vdim >> 2); idx += 256) {
+        const int e = idx << 2, g = e / p.vdim;
+        store4_as(v_row + (size_t)g * p.page_size * p.vdim + (e - g * p.vdim), load4_as(v_in + e));
+      }
+    const int per_warp = 32 / lanes, sub = lane / lanes, at = lane - sub * lanes;
+    for (int h0 = warp * per_warp; h0 < all_heads; h0 += WARPS * per_warp) {
+      const int head = h0 + sub;
+      const bool live = head < all_heads, is_q = head < p.heads;
+      const T* src = is_q ? q_in + (size_t)head * D : k_in + (size_t)(head - p.heads) * D;
+      const float* weight = is_q ? p.q_weight : p.k_weight;
+      float4 x[N], partner[N];
+      float sq = 0.f;
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        const int d = (n * lanes + at) << 2;
+        x[n] = partner[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (live && d < D) {
+          x[n] = load4_as(src + d);
+          if (!p.interleaved && d < p.rot) partner[n] = load4_as(src + (d < half ? d + half : d - half));
+        }
+        sq += fmaf(x[n].x, x[n].x, x[n].y * x[n].y) + fmaf(x[n].z, x[n].z, x[n].w * x[n].w);
+      }
+      float scale = 1.f;
+      if (p.q_weight != nullptr) {
+        for (int m = lanes >> 1; m > 0; m >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, m);
+        scale = 1.f / sqrtf(sq / (float)D + p.eps);
+      }
+      auto weighed = [&](float4 y, int d) {
+        y.x *= scale; y.y *= scale; y.z *= scale; y.w *= scale;
+        if (weight != nullptr) {
+          const float4 w = *reinterpret_cast<const float4*>(weight + d);
+          y.x *= w.x; y.y *= w.y; y.z *= w.z; y.w *= w.w;
+        }
+        return y;
+      };
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        const int d = (n * lanes + at) << 2;
+        if (!live || d >= D) continue;
+        float4 y = weighed(x[n], d);
+        if (d < p.rot) {
+          const float4 u = y;
+          if (p.interleaved) {
+            const float2 s = *reinterpret_cast<const float2*>(sine + (d >> 1)), c = *reinterpret_cast<const float2*>(cosine + (d >> 1));
+            rotate_pair(u.x, u.y, s.x, c.x, &y.x, &y.y);
+            rotate_pair(u.z, u.w, s.y, c.y, &y.z, &y.w);
+          } else {
+            const bool first = d < half;
+            const int i = first ? d : d - half;
+            const float4 v = weighed(partner[n], first ? d + half : i);
+            const float4 s = *reinterpret_cast<const float4*>(sine + i), c = *reinterpret_cast<const float4*>(cosine + i);
+            const float sign = first ? -1.f : 1.f;      // u cos - v sin, or (the second of a pair) v cos + u sin
+            y.x = __fadd_rn(__fmul_rn(u.x, c.x), sign * __fmul_rn(v.x, s.x));
+            y.y = __fadd_rn(__fmul_rn(u.y, c.y), sign * __fmul_rn(v.y, s.y));
+            y.z = __fadd_rn(__fmul_rn(u.z, c.z), sign * __fmul_rn(v.z, s.z));
+            y.w = __fadd_rn(__fmul_rn(u.w, c.w), sign * __fmul_rn(v.w, s.w));
+          }
+        }
+        if (is_q) store4_as(q_out + (size_t)head * D + d, y);
+        else store4_as(k_row + (size_t)(head - p.heads) * p.page_size * D + d, y);
+      }
+    }
+    return;
+  }
+
+  if (store)
+    for (int idx = threadIdx.x; idx < p.kv_heads * p.vdim; idx += 256) {
+      const int g = idx / p.vdim, d = idx - g * p.vdim;
+      v_row[(size_t)g * p.page_size * p.vdim + d] = v_in[idx];
+    }
+  for (int head = warp; head < all_heads; head += WARPS) {
+    const bool is_q = head < p.heads;
+    const T* src = is_q ? q_in + (size_t)head * D : k_in + (size_t)(head - p.heads) * D;
+    const float* weight = is_q ? p.q_weight : p.k_weight;
+    float scale = 1.f;
+    if (weight != nullptr) {
+      float sq = 0.f;
+      for (int d = lane; d < D; d += 32) sq = fmaf(to_float(src[d]), to_float(src[d]), sq);
+      scale = 1.f / sqrtf(warp_sum(sq) / (float)D + p.eps);
+    }
+    auto entry = [&](int d) { return to_float(src[d]) * scale * (weight != nullptr ? weight[d] : 1.f); };
+    T* dst = is_q ? q_out + (size_t)head * D : k_row + (size_t)(head - p.heads) * p.page_size * D;
+    for (int d = lane; d < D; d += 32) {
+      float y = entry(d);
+      if (d < p.rot) {
+        const bool first = p.interleaved ? (d & 1) == 0 : d < half;
+        const int i = p.interleaved ? d >> 1 : first ? d : d - half;
+        int a, b;
+        pair_places(i, p.rot, p.interleaved, &a, &b);
+        float y1, y2;
+        rotate_pair(entry(a), entry(b), sine[i], cosine[i], &y1, &y2);
+        y = first ? y1 : y2;
+      }
+      dst[d] = from_float<T>(y);
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 turn_heads_kernel(T* x, const int* positions, const float* __restrict__ freq, int heads, int dim, int n, int interleaved,
@@ -466,6 +617,48 @@ MLR_EXPORT int mlr_rotated_prepare(const float* qkv, const int* positions, const
   };
   if (dtype == MLR_F32) return launch_typed((float*)q_out, (float*)k_pool, (float*)v_pool);
   if (dtype == MLR_BF16) return launch_typed((bf16*)q_out, (bf16*)k_pool, (bf16*)v_pool);
+  return MLR_BAD_DTYPE;
+}
+
+// q, k, v: rows in `dtype` with row strides in entries; q_weight, k_weight: float32 [dim], both or neither; freq:
+// float32 [rot / 2]; slots: int64 [rows] (negative: not stored); q_out: [rows, heads * dim]; k_pool [pages, kv_heads,
+// page_size, dim], v_pool [pages, kv_heads, page_size, vdim].
+MLR_EXPORT int mlr_head_prepare(const void* q, long long q_stride, const void* k, long long k_stride, const void* v,
+                                long long v_stride, const int* positions, const float* q_weight, const float* k_weight,
+                                const float* freq, const long long* slots, void* q_out, void* k_pool, void* v_pool, int rows,
+                                int heads, int kv_heads, int dim, int vdim, int rot, int interleaved, float eps,
+                                float magnitude, int page_size, int write_kv, int dtype, cudaStream_t stream) {
+  if (rows == 0) return MLR_OK;
+  if (rows < 0 || heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || rot % 2 != 0 || page_size <= 0 ||
+      (rot > 0 && freq == nullptr) || (q_weight == nullptr) != (k_weight == nullptr))
+    return MLR_BAD_SIZE;
+  if (rot > 4096) return MLR_TOO_LARGE;
+  const HeadPrepareArgs p{q, k, v, q_stride, k_stride, v_stride, positions, q_weight, k_weight, freq, slots, q_out, k_pool,
+                          v_pool, heads, kv_heads, dim, vdim, rot, interleaved, page_size, write_kv, eps, magnitude};
+  const size_t piece = dtype == MLR_F32 ? 16 : 8;
+  auto aligned = [&](const void* ptr, size_t bytes) { return (reinterpret_cast<uintptr_t>(ptr) & (bytes - 1)) == 0; };
+  const bool pieces = dim % 4 == 0 && vdim % 4 == 0 && rot % (interleaved ? 4 : 8) == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 &&
+                      v_stride % 4 == 0 && dim <= 512 && aligned(q, piece) && aligned(k, piece) && aligned(v, piece) &&
+                      aligned(q_out, piece) && aligned(k_pool, piece) && aligned(v_pool, piece) && aligned(q_weight, 16) &&
+                      aligned(k_weight, 16);
+  int lanes = 1;
+  while (lanes < 32 && lanes * 4 < dim) lanes *= 2;
+  const int per_lane = (dim / 4 + lanes - 1) / lanes;
+  const size_t shared = sizeof(float) * (size_t)std::max(rot, 4);
+  auto launch = [&](auto kernel) {
+    launch_kernel(kernel, dim3(rows), dim3(256), shared, stream, p, lanes);
+    return launch_status();
+  };
+  if (dtype == MLR_F32) {
+    if (!pieces) return launch(head_prepare_kernel<float, 0>);
+    if (per_lane <= 1) return launch(head_prepare_kernel<float, 1>);
+    return per_lane <= 2 ? launch(head_prepare_kernel<float, 2>) : launch(head_prepare_kernel<float, 4>);
+  }
+  if (dtype == MLR_BF16) {
+    if (!pieces) return launch(head_prepare_kernel<bf16, 0>);
+    if (per_lane <= 1) return launch(head_prepare_kernel<bf16, 1>);
+    return per_lane <= 2 ? launch(head_prepare_kernel<bf16, 2>) : launch(head_prepare_kernel<bf16, 4>);
+  }
   return MLR_BAD_DTYPE;
 }
 

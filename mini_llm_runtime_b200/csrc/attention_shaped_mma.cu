@@ -1,12 +1,14 @@
-// Grouped-query softmax attention with shaped scores over keys that are also the values, on the tensor
-// cores (bfloat16, mma.sync m16n8k16).  Per head h, query position i and key position j:
+// Grouped-query softmax attention with shaped scores, on the tensor cores (bfloat16, mma.sync m16n8k16), over keys
+// that are also the values or over values of the keys' size of their own.  Per head h, query position i and key
+// position j:
 //
 //   x = softcap * tanh(q . k * scale / softcap)  (or q . k * scale without a cap)  - slope_h * (i - j)
 //   visible: j <= i, j in i's own chunk (chunk > 0), i - j < window (window > 0)
-//   out = sum_j e^x_j k_j / (sum_j e^x_j + e^sink_h), times sigmoid(gate) element by element
+//   out = sum_j e^x_j v_j / (sum_j e^x_j + e^sink_h), times sigmoid(gate) element by element
 //
 // Scores, cap, bias, softmax and sums are float32; the probabilities are rounded to bfloat16 for the second
-// product.  A key tile is fetched once and serves both products.
+// product.  Where keys are the values a key tile is fetched once and serves both products (OWN false); else a tile
+// of keys and one of values lie side by side in shared memory.
 //
 // shaped_prefill_kernel  work item (64 query rows of a segment, head): tiles of 64 keys aligned to absolute
 //                        positions, double-buffered with asynchronous copies, the tiles' places in the cache
@@ -35,6 +37,7 @@ struct ShapedArgs {
   const bf16* fresh; long long fresh_stride;     // decode: rows of kv_heads * D with the new keys, or null (already cached)
   const long long* slots;                        // decode with fresh: where each row's key goes
   bf16* pool;                                    // [pages, kv_heads, page_size, D]
+  const bf16* values;                            // the same for values of their own, or null
   bf16* out;                                     // [rows, heads * D]
   const bf16* gate; long long gate_stride;       // rows of heads * D, or null
   const float *slopes, *sinks;                   // [heads] or null
@@ -189,15 +192,15 @@ __device__ __forceinline__ int lowest_visible(const ShapedArgs& p, int position)
   return lo;
 }
 
-template <int D>
-__global__ void __launch_bounds__(ATTN_THREADS, D <= 64 ? 4 : 3)
+template <int D, bool OWN>
+__global__ void __launch_bounds__(ATTN_THREADS, OWN ? 2 : D <= 64 ? 4 : 3)
 shaped_prefill_kernel(const ShapedArgs p) {
   pdl_trigger();
   pdl_wait();
-  constexpr int PITCH = D + 8, PIECES = D / 8;
+  constexpr int PITCH = D + 8, PIECES = D / 8, KINDS = OWN ? 2 : 1, TILE = TILE_KV * PITCH;
   extern __shared__ __align__(128) uint8_t attn_shared[];
   bf16* q_tile = reinterpret_cast<bf16*>(attn_shared);         // [64][PITCH]
-  bf16* k_tiles = q_tile + TILE_Q * PITCH;                      // 2 x [64][PITCH]
+  bf16* k_tiles = q_tile + TILE_Q * PITCH;                      // 2 x [64][PITCH] (keys, then values of their own)
   __shared__ int places[2][TILE_KV];                            // pool rows of a tile's keys, two tiles ahead
 
   const int head = blockIdx.y, kv_head = head / (p.heads / p.kv_heads);
@@ -224,11 +227,12 @@ shaped_prefill_kernel(const ShapedArgs p) {
     }
   };
   auto fetch = [&](int t) {
-    bf16* tile = k_tiles + (t & 1) * TILE_KV * PITCH;
+    bf16* tile = k_tiles + (t & 1) * KINDS * TILE;
     for (int item = threadIdx.x; item < TILE_KV * PIECES; item += ATTN_THREADS) {
       const int r = item / PIECES, c = item - r * PIECES;
       const int row = places[t & 1][r];
       cp_async_16(tile + r * PITCH + c * 8, row >= 0 ? p.pool + (size_t)row * D + c * 8 : p.pool, row >= 0);
+      if (OWN) cp_async_16(tile + TILE + r * PITCH + c * 8, row >= 0 ? p.values + (size_t)row * D + c * 8 : p.values, row >= 0);
     }
     cp_async_commit();
   };
@@ -273,14 +277,14 @@ shaped_prefill_kernel(const ShapedArgs p) {
     }
     const int key0 = t * TILE_KV, key_last = key0 + TILE_KV - 1;
     if (warp_rows > 0 && key0 <= warp_last && key_last >= any_lo) {
-      const bf16* tile = k_tiles + (t & 1) * TILE_KV * PITCH;
+      const bf16* tile = k_tiles + (t & 1) * KINDS * TILE;
       float s[TILE_KV / 8][4];
       padded_qk<D, TILE_KV / 8>(s, q_frag, tile, lane);
       if (warp_rows == 16 && key_last <= warp_first && key0 >= all_lo)
         shaped_softmax_step<TILE_KV / 8, D / 8, false>(s, o, m, l, key0, position, limit_lo, slope2, p, lane);
       else
         shaped_softmax_step<TILE_KV / 8, D / 8, true>(s, o, m, l, key0, position, limit_lo, slope2, p, lane);
-      padded_pv<D, TILE_KV / 8>(o, s, tile, lane);
+      padded_pv<D, TILE_KV / 8>(o, s, tile + (KINDS - 1) * TILE, lane);
     }
     __syncthreads();
   }
@@ -313,22 +317,23 @@ shaped_prefill_kernel(const ShapedArgs p) {
 }
 
 constexpr int DEC_KEYS = 32;         // keys of a warp's tile
-constexpr int DEC_STAGES = 2;
+// tiles of a warp in shared memory: with values of their own and wide heads one, so that three blocks fit an SM
+template <int D, bool OWN> constexpr int DEC_STAGES = OWN && D > 64 ? 1 : 2;
 constexpr int DEC_ROWS = 16;         // query heads of one CTA
 constexpr int DEC_MAX_SPLITS = 64;
 constexpr int DEC_MIN_TILES = 4;     // key tiles a CTA takes at least (one per warp)
 
 // grid: (items, kv heads * blocks of 16 query heads, splits)
-template <int D>
+template <int D, bool OWN>
 __global__ void __launch_bounds__(ATTN_THREADS)
 shaped_decode_kernel(const ShapedArgs p) {
   pdl_trigger();
-  constexpr int PITCH = D + 8, PIECES = D / 8;
+  constexpr int PITCH = D + 8, PIECES = D / 8, KINDS = OWN ? 2 : 1, STAGES = DEC_STAGES<D, OWN>, TILE = DEC_KEYS * PITCH;
   constexpr int PER_LANE = DEC_KEYS * PIECES / 32;
   extern __shared__ __align__(128) uint8_t attn_shared[];
   bf16* q_tile = reinterpret_cast<bf16*>(attn_shared);                              // [16][PITCH]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  bf16* ring = q_tile + DEC_ROWS * PITCH + warp * DEC_STAGES * DEC_KEYS * PITCH;    // this warp's tiles
+  bf16* ring = q_tile + DEC_ROWS * PITCH + warp * STAGES * KINDS * TILE;            // this warp's tiles
   float* merged = reinterpret_cast<float*>(q_tile + DEC_ROWS * PITCH);              // [4][16][D] once the tiles are done
   __shared__ float warp_max_[ATTN_WARPS][DEC_ROWS], warp_sum_[ATTN_WARPS][DEC_ROWS];
   __shared__ int is_last;
@@ -367,13 +372,14 @@ shaped_decode_kernel(const ShapedArgs p) {
     return pool_row(p, table, key, kv_head);
   };
   auto fetch = [&](int place, int stage) {
-    bf16* tile = ring + stage * DEC_KEYS * PITCH;
+    bf16* tile = ring + stage * KINDS * TILE;
 #pragma unroll
     for (int i = 0; i < PER_LANE; ++i) {
       const int idx = i * 32 + lane, r = idx / PIECES, c = idx - r * PIECES;
       const int at = __shfl_sync(0xffffffffu, place, r);
       const bf16* src = at >= 0 ? p.pool + (size_t)at * D + c * 8 : at == -2 ? fresh + c * 8 : p.pool;
       cp_async_16(tile + r * PITCH + c * 8, src, at != -1);
+      if (OWN) cp_async_16(tile + TILE + r * PITCH + c * 8, at >= 0 ? p.values + (size_t)at * D + c * 8 : p.values, at >= 0);
     }
     cp_async_commit();
   };
@@ -402,8 +408,8 @@ shaped_decode_kernel(const ShapedArgs p) {
   for (int ks = 0; ks < D / 16; ++ks)
     ldmatrix_x4(q_frag[ks], q_tile + ((lane & 7) + (((lane >> 3) & 1) << 3)) * PITCH + (ks * 2 + (lane >> 4)) * 8);
   int stage = 0;
-  for (; tile < end; tile += ATTN_WARPS, stage ^= 1) {
-    if (tile + ATTN_WARPS < end) {
+  for (; tile < end; tile += ATTN_WARPS, stage = STAGES == 2 ? stage ^ 1 : 0) {
+    if (STAGES == 2 && tile + ATTN_WARPS < end) {
       fetch(next_place, stage ^ 1);
       next_place = look_up(tile + 2 * ATTN_WARPS);
       cp_async_wait<1>();
@@ -411,7 +417,7 @@ shaped_decode_kernel(const ShapedArgs p) {
       cp_async_wait<0>();
     }
     __syncwarp();
-    const bf16* keys = ring + stage * DEC_KEYS * PITCH;
+    const bf16* keys = ring + stage * KINDS * TILE;
     float s[DEC_KEYS / 8][4];
     padded_qk<D, DEC_KEYS / 8>(s, q_frag, keys, lane);
     const int key0 = tile * DEC_KEYS;
@@ -419,8 +425,12 @@ shaped_decode_kernel(const ShapedArgs p) {
       shaped_softmax_step<DEC_KEYS / 8, D / 8, false>(s, o, m, l, key0, position, limit_lo, slope2, p, lane);
     else
       shaped_softmax_step<DEC_KEYS / 8, D / 8, true>(s, o, m, l, key0, position, limit_lo, slope2, p, lane);
-    padded_pv<D, DEC_KEYS / 8>(o, s, keys, lane);
+    padded_pv<D, DEC_KEYS / 8>(o, s, keys + (KINDS - 1) * TILE, lane);
     __syncwarp();                                    // the next copies go into this tile
+    if (STAGES == 1 && tile + ATTN_WARPS < end) {
+      fetch(next_place, 0);
+      next_place = look_up(tile + 2 * ATTN_WARPS);
+    }
   }
 
   // the warps' parts, in the order of the warps
@@ -527,30 +537,37 @@ shaped_decode_kernel(const ShapedArgs p) {
   }
 }
 
-template <int D>
+template <int D, bool OWN>
 static int launch_shaped_prefill(const ShapedArgs& p, int tiles, cudaStream_t stream) {
-  const size_t shared = sizeof(bf16) * (size_t)(TILE_Q + 2 * TILE_KV) * (D + 8);
+  const size_t shared = sizeof(bf16) * (size_t)(TILE_Q + (OWN ? 4 : 2) * TILE_KV) * (D + 8);
   if (shared > 48 * 1024) {
-    cudaError_t err = cudaFuncSetAttribute(shaped_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+    cudaError_t err = cudaFuncSetAttribute(shaped_prefill_kernel<D, OWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
     if (err != cudaSuccess) return (int)err;
   }
-  launch_kernel(shaped_prefill_kernel<D>, dim3(tiles, p.heads), dim3(ATTN_THREADS), shared, stream, p);
+  launch_kernel(shaped_prefill_kernel<D, OWN>, dim3(tiles, p.heads), dim3(ATTN_THREADS), shared, stream, p);
+  return launch_status();
+}
+
+template <int D, bool OWN>
+static int launch_shaped_decode(const ShapedArgs& p, int items, cudaStream_t stream) {
+  const size_t tiles = sizeof(bf16) * (size_t)ATTN_WARPS * DEC_STAGES<D, OWN> * (OWN ? 2 : 1) * DEC_KEYS * (D + 8);
+  const size_t parts = sizeof(float) * (size_t)ATTN_WARPS * DEC_ROWS * D;
+  const size_t shared = sizeof(bf16) * (size_t)DEC_ROWS * (D + 8) + (tiles > parts ? tiles : parts);
+  if (shared > 48 * 1024) {
+    cudaError_t err = cudaFuncSetAttribute(shaped_decode_kernel<D, OWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+    if (err != cudaSuccess) return (int)err;
+  }
+  const int per = p.heads / p.kv_heads;
+  launch_kernel(shaped_decode_kernel<D, OWN>, dim3(items, p.kv_heads * ((per + DEC_ROWS - 1) / DEC_ROWS), p.splits),
+                dim3(ATTN_THREADS), shared, stream, p);
   return launch_status();
 }
 
 template <int D>
-static int launch_shaped_decode(const ShapedArgs& p, int items, cudaStream_t stream) {
-  const size_t tiles = sizeof(bf16) * (size_t)ATTN_WARPS * DEC_STAGES * DEC_KEYS * (D + 8);
-  const size_t parts = sizeof(float) * (size_t)ATTN_WARPS * DEC_ROWS * D;
-  const size_t shared = sizeof(bf16) * (size_t)DEC_ROWS * (D + 8) + (tiles > parts ? tiles : parts);
-  if (shared > 48 * 1024) {
-    cudaError_t err = cudaFuncSetAttribute(shaped_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
-    if (err != cudaSuccess) return (int)err;
-  }
-  const int per = p.heads / p.kv_heads;
-  launch_kernel(shaped_decode_kernel<D>, dim3(items, p.kv_heads * ((per + DEC_ROWS - 1) / DEC_ROWS), p.splits),
-                dim3(ATTN_THREADS), shared, stream, p);
-  return launch_status();
+static int launch_shaped(const ShapedArgs& p, int decode, int count, cudaStream_t stream) {
+  if (p.values != nullptr)
+    return decode ? launch_shaped_decode<D, true>(p, count, stream) : launch_shaped_prefill<D, true>(p, count, stream);
+  return decode ? launch_shaped_decode<D, false>(p, count, stream) : launch_shaped_prefill<D, false>(p, count, stream);
 }
 
 }  // namespace mlr
@@ -567,11 +584,12 @@ MLR_EXPORT int mlr_attention_shaped_mma_fits(int dim) { return dim == 32 || dim 
 // `splits` CTAs; partial: float32 [count, splits, heads, dim + 2] and counters: `count` * kv_heads * blocks of 16
 // heads zeros (left zero), both only with splits > 1.
 // q, gate, fresh: bfloat16 rows with strides (in elements); gate null: no gate; fresh null: the new keys are in
-// the pool already, else `slots` (int64 per row) says where they go.  softcap 0: no cap; slopes, sinks: float32
+// the pool already, else `slots` (int64 per row) says where they go (only where keys are the values: values null; else
+// values [pages, kv_heads, page_size, dim]).  softcap 0: no cap; slopes, sinks: float32
 // [heads] or null; chunk, window 0: none.
 MLR_EXPORT int mlr_attention_shaped_mma(int decode, const void* q, long long q_stride, const void* fresh,
-                                        long long fresh_stride, const long long* slots, void* pool, void* out,
-                                        const void* gate, long long gate_stride, const float* slopes, const float* sinks,
+                                        long long fresh_stride, const long long* slots, void* pool, const void* values,
+                                        void* out, const void* gate, long long gate_stride, const float* slopes, const float* sinks,
                                         const int* list_a, const int* list_b, int count, const int* seg_q_start,
                                         const int* seg_q_len, const int* seg_pos0, const int* block_table,
                                         const int* seg_slot, int table_width, int heads, int kv_heads, int dim,
@@ -579,18 +597,18 @@ MLR_EXPORT int mlr_attention_shaped_mma(int decode, const void* q, long long q_s
                                         int* counters, int splits, cudaStream_t stream) {
   if (count == 0) return MLR_OK;
   if (count < 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || page_size <= 0 || table_width <= 0 ||
-      window < 0 || chunk < 0 || softcap < 0.f || splits < 1 || (fresh != nullptr && slots == nullptr) ||
+      window < 0 || chunk < 0 || softcap < 0.f || splits < 1 || (fresh != nullptr && (slots == nullptr || values != nullptr)) ||
       (splits > 1 && (partial == nullptr || counters == nullptr)))
     return MLR_BAD_SIZE;
   auto aligned = [](const void* ptr) { return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0; };
-  if (!aligned(q) || !aligned(fresh) || !aligned(pool) || !aligned(out) || q_stride % 8 || fresh_stride % 8 ||
+  if (!aligned(q) || !aligned(fresh) || !aligned(pool) || !aligned(values) || !aligned(out) || q_stride % 8 || fresh_stride % 8 ||
       gate_stride % 2 || (reinterpret_cast<uintptr_t>(gate) & 3))
     return MLR_BAD_ALIGNMENT;
   if (heads > 65535 || splits > DEC_MAX_SPLITS) return MLR_TOO_LARGE;
   ShapedArgs p;
   p.q = (const bf16*)q; p.q_stride = q_stride;
   p.fresh = (const bf16*)fresh; p.fresh_stride = fresh_stride; p.slots = slots;
-  p.pool = (bf16*)pool; p.out = (bf16*)out; p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
+  p.pool = (bf16*)pool; p.values = (const bf16*)values; p.out = (bf16*)out; p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
   p.slopes = slopes; p.sinks = sinks;
   p.tile_seg = list_a; p.tile_row0 = list_b; p.decode_seg = list_a;
   p.seg_q_start = seg_q_start; p.seg_q_len = seg_q_len; p.seg_pos0 = seg_pos0;
@@ -607,10 +625,10 @@ MLR_EXPORT int mlr_attention_shaped_mma(int decode, const void* q, long long q_s
   p.limits = partial == nullptr ? nullptr : reinterpret_cast<float2*>(partial + (size_t)count * splits * heads * dim);
   p.counters = counters; p.splits = splits;
   switch (dim) {
-    case 32: return decode ? launch_shaped_decode<32>(p, count, stream) : launch_shaped_prefill<32>(p, count, stream);
-    case 64: return decode ? launch_shaped_decode<64>(p, count, stream) : launch_shaped_prefill<64>(p, count, stream);
-    case 96: return decode ? launch_shaped_decode<96>(p, count, stream) : launch_shaped_prefill<96>(p, count, stream);
-    case 128: return decode ? launch_shaped_decode<128>(p, count, stream) : launch_shaped_prefill<128>(p, count, stream);
+    case 32: return launch_shaped<32>(p, decode, count, stream);
+    case 64: return launch_shaped<64>(p, decode, count, stream);
+    case 96: return launch_shaped<96>(p, decode, count, stream);
+    case 128: return launch_shaped<128>(p, decode, count, stream);
     default: return MLR_BAD_SIZE;
   }
 }

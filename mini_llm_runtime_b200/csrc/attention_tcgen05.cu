@@ -791,14 +791,15 @@ MLR_EXPORT int mlr_attention_prefill_tcgen05(const void* q, const void* k_pool, 
                         scale, max_kv_len, queue, error_word, scratch, scratch_bytes, counters, counters_len, stream);
 }
 
-// The same with shaped scores over keys that are also the values (pool: [pool_pages, kv_heads, page_size,
-// head_dim]).  q: rows spaced q_stride apart (a multiple of 8), starting at the row's first column; softcap 0: no
+// The same with shaped scores (pools: [pool_pages, kv_heads, page_size, head_dim]; keys that are also the values: one
+// pool twice).  q: rows spaced q_stride apart (a multiple of 8), starting at the row's first column; softcap 0: no
 // cap; slopes, sinks: float32 [heads] or null; chunk, window 0: none; gate: bfloat16 rows of heads * head_dim
 // entries spaced gate_stride apart (even), or null.
 MLR_EXPORT int mlr_attention_shaped_prefill_tcgen05(
-    const void* q, long long q_stride, const void* pool, void* out, const int* tile_seg, const int* tile_row0,
-    const int* seg_q_start, const int* seg_q_len, const int* seg_pos0, const int* block_table, const int* seg_slot,
-    int table_width, int tiles, int q_rows, int heads, int kv_heads, int head_dim, int page_size, int pool_pages, int window,
+    const void* q, long long q_stride, const void* k_pool, const void* v_pool, void* out, const int* tile_seg,
+    const int* tile_row0, const int* seg_q_start, const int* seg_q_len, const int* seg_pos0, const int* block_table,
+    const int* seg_slot, int table_width, int tiles, int q_rows, int heads, int kv_heads, int head_dim, int page_size,
+    int pool_pages, int window,
     int chunk, float scale, float softcap, const float* slopes, const float* sinks, const void* gate, long long gate_stride,
     int max_kv_len, int* queue, int* error_word, void* scratch, long long scratch_bytes, int* counters, int counters_len,
     cudaStream_t stream) {
@@ -811,7 +812,7 @@ MLR_EXPORT int mlr_attention_shaped_prefill_tcgen05(
   if ((long long)tiles * heads >= (1ll << 30)) return MLR_TOO_LARGE;
   const int page_shift = fa_shift_of(page_size);
   if (page_shift < 3) return MLR_BAD_SIZE;
-  if (((uintptr_t)pool & 15) || ((uintptr_t)q & 15) || q_stride % 8 || ((uintptr_t)gate & 3) || gate_stride % 2)
+  if (((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15) || ((uintptr_t)q & 15) || q_stride % 8 || ((uintptr_t)gate & 3) || gate_stride % 2)
     return MLR_BAD_ALIGNMENT;
   const long long pool_rows = (long long)pool_pages * kv_heads * page_size;
   if (pool_rows >= (1ll << 31)) return MLR_TOO_LARGE;
@@ -826,11 +827,11 @@ MLR_EXPORT int mlr_attention_shaped_prefill_tcgen05(
   score.gate = (const bf16*)gate;
   score.gate_stride = gate_stride;
   if (head_dim == 64)
-    return fa_launch<64, true>(q, pool, pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot,
+    return fa_launch<64, true>(q, k_pool, v_pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot,
                                table_width, tiles, q_rows, heads, kv_heads, page_size, page_shift, pool_rows, window, scale,
                                max_kv_len, queue, error_word, scratch, scratch_bytes, counters, counters_len, stream, q_stride,
                                score);
-  return fa_launch<128, true>(q, pool, pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot,
+  return fa_launch<128, true>(q, k_pool, v_pool, out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot,
                               table_width, tiles, q_rows, heads, kv_heads, page_size, page_shift, pool_rows, window, scale,
                               max_kv_len, queue, error_word, scratch, scratch_bytes, counters, counters_len, stream, q_stride,
                               score);

@@ -237,6 +237,14 @@ __device__ __forceinline__ void reduce_swapped_swiglu(const float* partials, int
   const int n0 = tile_x * 64 + 4 * rg;
   if (n0 >= half) return;
   const bool wide = (half & 3) == 0;
+  float gate_bias[4] = {0.f, 0.f, 0.f, 0.f}, up_bias[4] = {0.f, 0.f, 0.f, 0.f};
+  if (p.bias != nullptr) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      gate_bias[e] = to_float(p.bias[tile_x * TILE_ROWS + 4 * rg + e]);
+      up_bias[e] = to_float(p.bias[tile_x * TILE_ROWS + 64 + 4 * rg + e]);
+    }
+  }
   constexpr int CB = 2;
   for (int c = cg; c < BN; c += 8 * CB) {
     float4 gate[CB], up[CB];
@@ -266,8 +274,11 @@ __device__ __forceinline__ void reduce_swapped_swiglu(const float* partials, int
     for (int j = 0; j < CB; ++j) {
       const int col = c + 8 * j, m = b_row0 + col;
       if (col >= BN || m >= p.M) continue;
-      const float v[4] = {gate_times(p.gate_act, gate[j].x, up[j].x, p.gate_limit, p.gate_slope), gate_times(p.gate_act, gate[j].y, up[j].y, p.gate_limit, p.gate_slope),
-                          gate_times(p.gate_act, gate[j].z, up[j].z, p.gate_limit, p.gate_slope), gate_times(p.gate_act, gate[j].w, up[j].w, p.gate_limit, p.gate_slope)};
+      const float g[4] = {gate[j].x + gate_bias[0], gate[j].y + gate_bias[1], gate[j].z + gate_bias[2], gate[j].w + gate_bias[3]};
+      const float u[4] = {up[j].x + up_bias[0], up[j].y + up_bias[1], up[j].z + up_bias[2], up[j].w + up_bias[3]};
+      float v[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = gate_times(p.gate_act, g[e], u[e], p.gate_limit, p.gate_slope);
       bf16* dst = (bf16*)p.out + (size_t)m * half + n0;
       if (wide) {
         __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
@@ -508,6 +519,24 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             for (int c = 0; c < 32; ++c) {
               g[c] = __float_as_uint(scale * __uint_as_float(g[c]));
               u[c] = __float_as_uint(scale * __uint_as_float(u[c]));
+            }
+          }
+          if (p.bias != nullptr) {
+            const uint4* gate_bias = reinterpret_cast<const uint4*>(p.bias + (tile_y * (BN / 128) + block) * 128 + c0);
+#pragma unroll
+            for (int piece = 0; piece < 4; ++piece) {
+              const uint4 bg = gate_bias[piece], bu = gate_bias[piece + 8];      // 64 entries on: the up bias
+              const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&bg);
+              const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&bu);
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const float2 gf = __bfloat1622float2(g2[e]), uf = __bfloat1622float2(u2[e]);
+                const int c = piece * 8 + 2 * e;
+                g[c] = __float_as_uint(__uint_as_float(g[c]) + gf.x);
+                g[c + 1] = __float_as_uint(__uint_as_float(g[c + 1]) + gf.y);
+                u[c] = __float_as_uint(__uint_as_float(u[c]) + uf.x);
+                u[c + 1] = __float_as_uint(__uint_as_float(u[c + 1]) + uf.y);
+              }
             }
           }
 #pragma unroll
@@ -835,7 +864,7 @@ MLR_EXPORT long long mlr_gemm_tcgen05_plan(int M, int N, int K, int swiglu, int*
 // result is act(gate) * up, act being silu (swiglu == 1) or the tanh form of gelu (swiglu == 2), or
 // (swiglu == 3) the clamped gate g * sigmoid(gate_slope * g) * (u + 1) with g = min(gate, gate_limit) and
 // u = clamp(up, -gate_limit, gate_limit)
-// (N % 128 == 0, no bias) and out is silu(gate) * up, [M, N/2] bfloat16.
+// (N % 128 == 0; the bias comes first) and out is act(gate) * up, [M, N/2] bfloat16.
 // scratch: at least mlr_gemm_tcgen05_plan(...) bytes; counters: one zeroed int per tile;
 // error_word: host-visible int that receives a non-zero code if a wait inside the kernel runs out.
 MLR_EXPORT int mlr_gemm_tcgen05(const void* x, const void* w, const void* bias, void* out, int M, int N, int K,
@@ -844,7 +873,8 @@ MLR_EXPORT int mlr_gemm_tcgen05(const void* x, const void* w, const void* bias, 
   if (M == 0) return MLR_OK;
   if (M < 0 || N <= 0 || K <= 0) return MLR_BAD_SIZE;
   if (K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return MLR_BAD_ALIGNMENT;
-  if (swiglu && (N % 128 != 0 || bias != nullptr || out_f32)) return MLR_BAD_SIZE;
+  if (swiglu && (N % 128 != 0 || out_f32)) return MLR_BAD_SIZE;
+  if ((uintptr_t)bias & (swiglu ? 15 : 1)) return MLR_BAD_ALIGNMENT;
   const GemmPlan plan = plan_gemm(M, N, K, swiglu != 0);
   GemmParams p;
   p.M = M; p.N = N; p.K = K;

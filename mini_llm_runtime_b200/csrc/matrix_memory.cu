@@ -1,0 +1,510 @@
+// A matrix memory with exponential gates (the mLSTM of xLSTM): per request and head a memory S [dim, vdim] and a
+// normaliser n [dim] in 32-bit floats that are carried from token to token,
+//
+//   i = cap tanh((i_raw + i_bias) / cap),   f = logsigmoid(cap tanh((f_raw + f_bias) / cap))       (logarithms)
+//   m_t = max(f + m_{t-1}, i)
+//   S_t = e^(f + m_{t-1} - m_t) S_{t-1} + e^(i - m_t) k_t v_t^T,      n_t likewise with k_t alone
+//   o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + guard),           q = q_raw * dim^-1/2
+//   out = o / rms(o) * weight * sigmoid(gate)                          (rms over a head's channels)
+//
+// The state is kept transposed with n as one more value channel (whose value is 1): [vdim + 1, dim].
+//
+// matrix_memory_decode_kernel   steps of single rows: everything above in one launch, a block per (request, head).
+// matrix_memory_gates_kernel    per token and head [keep, write, e^(-m)]: the running maximum is an associative scan of
+//                               maps m -> max(a + m, b).  Wherever m appears the same rounded m_t is used, so what m's
+//                               own rounding does to S cancels out.
+// matrix_memory_scan_kernel     the recurrence of longer segments, token after token, value channels over blocks.
+// matrix_memory_finish_kernel   normaliser, head norm, weight and gate of the scan's rows.
+#include "common.cuh"
+#include "copy_async.cuh"
+#include "lane_sums.cuh"
+
+namespace mlr {
+
+struct MemoryArgs {
+  const float *q, *k, *v, *i_raw, *f_raw, *gate;      // row-major views, one row per token
+  long long q_stride, k_stride, v_stride, i_stride, f_stride, gate_stride;
+  const float *i_bias, *f_bias;         // [heads]
+  const float* weight;                  // [heads * vdim]
+  float4* coef;                         // [rows, heads]: keep, write, e^(-m), unused
+  float* reads;                         // [rows, heads, vdim]: S^T q before the normaliser
+  float* norms;                         // [rows, heads]: n . q
+  float* states;                        // [slots, heads, vdim + 1, dim]
+  float* maxima;                        // [slots, heads]
+  const int *seg_q_start, *seg_q_len, *seg_slot;
+  int heads, dim, vdim;
+  float cap, guard, eps, q_scale;
+};
+
+__device__ __forceinline__ float capped(float raw, float cap) { return cap * tanhf(raw / cap); }
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// ------------------------------------------------------------------ single rows
+constexpr int DECODE_THREADS = 256;
+constexpr int DECODE_WARPS = DECODE_THREADS / 32;
+
+// PIECES: 16-byte pieces of a state row per lane (dim <= 128 * PIECES, rows and pointers aligned), or 0: any
+// size, number by number.  grid: (segments, heads).
+template <typename T, int PIECES>
+__global__ void __launch_bounds__(DECODE_THREADS)
+matrix_memory_decode_kernel(MemoryArgs p, T* __restrict__ out) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float shared[];      // [vdim + 1] reads
+  __shared__ float scratch[32];
+  const int seg = blockIdx.x, head = blockIdx.y, D = p.dim, V = p.vdim;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const size_t slot_head = (size_t)p.seg_slot[seg] * p.heads + head;
+  const size_t row = p.seg_q_start[seg];
+  float* state = p.states + slot_head * (size_t)(V + 1) * D;
+  const float i_bias = p.i_bias[head], f_bias = p.f_bias[head];
+  pdl_wait();
+  const float i_raw = __ldcg(p.i_raw + row * p.i_stride + head), f_raw = __ldcg(p.f_raw + row * p.f_stride + head);
+  const float m_old = __ldcg(p.maxima + slot_head);
+  const float* q = p.q + row * p.q_stride + (size_t)head * D;
+  const float* k = p.k + row * p.k_stride + (size_t)head * D;
+  const float* v = p.v + row * p.v_stride + (size_t)head * V;
+  float m_new = 0.f, keep = 0.f, write = 0.f;
+  auto gates = [&]() {
+    const float log_in = capped(i_raw + i_bias, p.cap), log_forget = log_sigmoid(capped(f_raw + f_bias, p.cap));
+    m_new = fmaxf(log_forget + m_old, log_in);
+    keep = expf(log_forget + m_old - m_new);
+    write = expf(log_in - m_new);
+  };
+  if (PIECES > 0) {
+    constexpr int N = PIECES > 0 ? PIECES : 1, ROWS = N >= 4 ? 2 : 8 / N;      // state rows in flight per warp
+    float4 q4[N], k4[N];
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int d = (n * 32 + lane) << 2;
+      q4[n] = k4[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < D) {
+        q4[n] = __ldcg(reinterpret_cast<const float4*>(q + d));
+        k4[n] = __ldcg(reinterpret_cast<const float4*>(k + d));
+      }
+    }
+    bool first = true;
+    for (int v0 = warp; v0 <= V; v0 += DECODE_WARPS * ROWS) {
+      float4 s[ROWS][N];
+      float value[ROWS], sum[ROWS];
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        const int c = v0 + r * DECODE_WARPS;
+        value[r] = c < V ? __ldcg(v + c) : 1.f;
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+          const int d = (n * 32 + lane) << 2;
+          s[r][n] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (c <= V && d < D) s[r][n] = __ldcg(reinterpret_cast<const float4*>(state + (size_t)c * D + d));
+        }
+      }
+      if (first) gates();      // while the state is on its way
+      first = false;
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        const int c = v0 + r * DECODE_WARPS;
+        const float u = write * value[r];
+        sum[r] = 0.f;
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+          const int d = (n * 32 + lane) << 2;
+          float4& x = s[r][n];
+          x.x = fmaf(k4[n].x, u, keep * x.x); x.y = fmaf(k4[n].y, u, keep * x.y);
+          x.z = fmaf(k4[n].z, u, keep * x.z); x.w = fmaf(k4[n].w, u, keep * x.w);
+          sum[r] = fmaf(q4[n].x, x.x, sum[r]); sum[r] = fmaf(q4[n].y, x.y, sum[r]);
+          sum[r] = fmaf(q4[n].z, x.z, sum[r]); sum[r] = fmaf(q4[n].w, x.w, sum[r]);
+          if (c <= V && d < D) *reinterpret_cast<float4*>(state + (size_t)c * D + d) = x;
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) sum[r] = warp_sum(sum[r]);
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        const int c = v0 + r * DECODE_WARPS;
+        if (lane == 0 && c <= V) shared[c] = sum[r] * p.q_scale;
+      }
+    }
+    if (first) gates();        // a warp without a row of its own
+  } else {
+    gates();
+    for (int c = warp; c <= V; c += DECODE_WARPS) {
+      const float u = write * (c < V ? __ldcg(v + c) : 1.f);
+      float sum = 0.f;
+      for (int d = lane; d < D; d += 32) {
+        float* s = state + (size_t)c * D + d;
+        const float x = fmaf(__ldcg(k + d), u, keep * __ldcg(s));
+        *s = x;
+        sum = fmaf(__ldcg(q + d), x, sum);
+      }
+      sum = warp_sum(sum);
+      if (lane == 0) shared[c] = sum * p.q_scale;
+    }
+  }
+  __syncthreads();
+  if (threadIdx.x == 0) p.maxima[slot_head] = m_new;      // every thread read the old one before the barrier
+  const float inverse = 1.f / (fmaxf(fabsf(shared[V]), expf(-m_new)) + p.guard);
+  float sq = 0.f;
+  for (int c = threadIdx.x; c < V; c += DECODE_THREADS) {
+    const float o = shared[c] * inverse;
+    sq = fmaf(o, o, sq);
+  }
+  const float factor = inverse / sqrtf(block_sum(sq, scratch) / (float)V + p.eps);
+  for (int c = threadIdx.x; c < V; c += DECODE_THREADS) {
+    const float g = __ldcg(p.gate + row * p.gate_stride + (size_t)head * V + c);
+    out[row * p.heads * V + (size_t)head * V + c] = from_float<T>(shared[c] * factor * p.weight[head * V + c] * sigmoid(g));
+  }
+}
+
+// ------------------------------------------------------------------ gates of longer segments
+constexpr int GATE_THREADS = 256;
+constexpr int GATE_WARPS = GATE_THREADS / 32;
+
+// grid: (segments, heads).  256 tokens per turn.
+__global__ void __launch_bounds__(GATE_THREADS)
+matrix_memory_gates_kernel(MemoryArgs p) {
+  __shared__ float total_a[GATE_WARPS], total_b[GATE_WARPS], last[GATE_WARPS];
+  const int seg = blockIdx.x, head = blockIdx.y;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const size_t slot_head = (size_t)p.seg_slot[seg] * p.heads + head;
+  const size_t row0 = p.seg_q_start[seg];
+  const int q_len = p.seg_q_len[seg];
+  const float i_bias = p.i_bias[head], f_bias = p.f_bias[head];
+  // The recurrence behind this kernel is few blocks that run long: brought in while the product in front of this
+  // kernel still fills the SMs, they would land several to an SM.  So the trigger comes after the wait.
+  pdl_wait();
+  pdl_trigger();
+  float before = __ldcg(p.maxima + slot_head);       // m ahead of this turn's tokens
+  float i_next = 0.f, f_next = 0.f;
+  auto ask = [&](int t) {
+    if (t < q_len) {
+      i_next = __ldcg(p.i_raw + (row0 + t) * p.i_stride + head);
+      f_next = __ldcg(p.f_raw + (row0 + t) * p.f_stride + head);
+    }
+  };
+  ask(threadIdx.x);
+  for (int t0 = 0; t0 < q_len; t0 += GATE_THREADS) {
+    const int t = t0 + threadIdx.x;
+    float log_in = -INFINITY, log_forget = 0.f;      // a place without a token changes nothing
+    if (t < q_len) {
+      log_in = capped(i_next + i_bias, p.cap);
+      log_forget = log_sigmoid(capped(f_next + f_bias, p.cap));
+    }
+    ask(t + GATE_THREADS);
+    // inclusive scan of the maps m -> max(a + m, b), earlier tokens first
+    float a = log_forget, b = log_in;
+#pragma unroll
+    for (int step = 1; step < 32; step <<= 1) {
+      const float a_up = __shfl_up_sync(0xffffffffu, a, step), b_up = __shfl_up_sync(0xffffffffu, b, step);
+      if (lane >= step) {
+        b = fmaxf(b_up + a, b);
+        a += a_up;
+      }
+    }
+    if (lane == 31) {
+      total_a[warp] = a;
+      total_b[warp] = b;
+    }
+    __syncthreads();
+    float carried = before;
+    for (int w = 0; w < warp; ++w) carried = fmaxf(total_a[w] + carried, total_b[w]);
+    const float m = fmaxf(a + carried, b);
+    if (lane == 31) last[warp] = m;
+    __syncthreads();
+    float m_before = __shfl_up_sync(0xffffffffu, m, 1);
+    if (lane == 0) m_before = warp > 0 ? last[warp - 1] : before;
+    if (t < q_len)
+      p.coef[(row0 + t) * p.heads + head] = make_float4(expf(log_forget + m_before - m), expf(log_in - m), expf(-m), 0.f);
+    before = last[GATE_WARPS - 1];
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) p.maxima[slot_head] = before;
+}
+
+// ------------------------------------------------------------------ the recurrence of longer segments
+// grid: (segments, heads, blocks of state rows).  A group of SL lanes holds C rows of the head's transposed state
+// (value channels, the last one the normaliser's), each lane E key channels of them in interleaved pieces of four.
+// Reads are summed over the lanes for TB tokens at once; the updates need no sum.  WIDE: rows are staged in 16-byte
+// pieces (sizes and strides multiples of four floats, pointers aligned).
+template <int E, int SL, int C, bool WIDE, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+matrix_memory_scan_kernel(MemoryArgs p) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float shared[];
+  constexpr int TB = 4, GROUPS = THREADS / SL, COLS = GROUPS * C, N = TB * C;
+  constexpr int TOKENS = SL == 32 ? 16 : 32;      // tokens staged at once
+  constexpr int pitch = E * SL;                   // staged rows of keys and queries, filled up with zeros
+  constexpr int COEF = 4;
+  constexpr int buffer = TOKENS * (2 * pitch + COLS + COEF);
+  const int D = p.dim, V = p.vdim;
+  const int seg = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS;
+  const int lane = threadIdx.x & 31, s = threadIdx.x % SL, group = threadIdx.x / SL;
+  const int q_start = p.seg_q_start[seg], q_len = p.seg_q_len[seg];
+  float* state = p.states + ((size_t)p.seg_slot[seg] * p.heads + head) * (size_t)(V + 1) * D;
+
+  // what no copy overwrites: zeros behind the rows' D entries, the normaliser's value of one, zeros behind it
+  if (D < pitch) {
+    for (int idx = threadIdx.x; idx < 4 * TOKENS * (pitch - D); idx += THREADS) {
+      const int r = idx / (pitch - D), d = D + idx - r * (pitch - D);
+      shared[(r / (2 * TOKENS)) * buffer + (r % (2 * TOKENS)) * pitch + d] = 0.f;
+    }
+  }
+  if (col0 + COLS > V) {
+    for (int idx = threadIdx.x; idx < 2 * TOKENS * COLS; idx += THREADS) {
+      const int which = idx / (TOKENS * COLS), at = idx - which * TOKENS * COLS, c = at % COLS;
+      if (col0 + c >= V) shared[which * buffer + 2 * TOKENS * pitch + at] = col0 + c == V ? 1.f : 0.f;
+    }
+  }
+  pdl_wait();
+  auto stage = [&](int t0, int which) {
+    float* k_rows = shared + which * buffer;
+    float* q_rows = k_rows + TOKENS * pitch;
+    float* v_rows = q_rows + TOKENS * pitch;
+    float* coef = v_rows + TOKENS * COLS;
+    const int tokens = min(TOKENS, q_len - t0);
+    const size_t row0 = (size_t)(q_start + t0);
+    if (WIDE) {
+      const int per_row = D >> 2;
+      for (int idx = threadIdx.x; idx < tokens * per_row; idx += THREADS) {
+        const int t = idx / per_row, d = (idx - t * per_row) << 2;
+        copy_async_16(k_rows + t * pitch + d, p.k + (row0 + t) * p.k_stride + (size_t)head * D + d);
+        copy_async_16(q_rows + t * pitch + d, p.q + (row0 + t) * p.q_stride + (size_t)head * D + d);
+      }
+      constexpr int V_PIECES = (COLS + 3) / 4;
+      for (int idx = threadIdx.x; idx < tokens * V_PIECES; idx += THREADS) {
+        const int t = idx / V_PIECES, c = (idx - t * V_PIECES) << 2;
+        if (col0 + c < V) copy_async_16(v_rows + t * COLS + c, p.v + (row0 + t) * p.v_stride + (size_t)head * V + col0 + c);
+      }
+    } else {
+      for (int idx = threadIdx.x; idx < tokens * D; idx += THREADS) {
+        const int t = idx / D, d = idx - t * D;
+        copy_async_4(k_rows + t * pitch + d, p.k + (row0 + t) * p.k_stride + (size_t)head * D + d);
+        copy_async_4(q_rows + t * pitch + d, p.q + (row0 + t) * p.q_stride + (size_t)head * D + d);
+      }
+      for (int idx = threadIdx.x; idx < tokens * COLS; idx += THREADS) {
+        const int t = idx / COLS, c = idx - t * COLS;
+        if (col0 + c < V) copy_async_4(v_rows + idx, p.v + (row0 + t) * p.v_stride + (size_t)head * V + col0 + c);
+      }
+    }
+    if (threadIdx.x < tokens)
+      copy_async_16(coef + threadIdx.x * COEF, reinterpret_cast<const float*>(p.coef + (row0 + threadIdx.x) * p.heads + head));
+    copy_async_commit();
+    if (tokens % TB != 0) {      // the rest of the last block of tokens: kept as it is, nothing written
+      const int fill = TB - tokens % TB;
+      for (int idx = threadIdx.x; idx < fill * pitch; idx += THREADS) k_rows[tokens * pitch + idx] = q_rows[tokens * pitch + idx] = 0.f;
+      for (int idx = threadIdx.x; idx < fill * COLS; idx += THREADS) v_rows[tokens * COLS + idx] = 0.f;
+      for (int idx = threadIdx.x; idx < fill * COEF; idx += THREADS) coef[tokens * COEF + idx] = idx % COEF == 0 ? 1.f : 0.f;
+    }
+  };
+  stage(0, 0);
+  auto entry = [&](int i) { return (((i >> 2) * SL + s) << 2) + (i & 3); };      // key channel of a lane's i-th number
+  float S[C][E];
+#pragma unroll
+  for (int c = 0; c < C; ++c) {
+    const int column = col0 + group * C + c;
+    const bool mine = column <= V;
+    const float* src = state + (size_t)(mine ? column : 0) * D;
+    if (WIDE) {
+#pragma unroll
+      for (int i = 0; i < E; i += 4) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (mine && entry(i) < D) x = __ldcg(reinterpret_cast<const float4*>(src + entry(i)));
+        S[c][i] = x.x; S[c][i + 1] = x.y; S[c][i + 2] = x.z; S[c][i + 3] = x.w;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < E; ++i) S[c][i] = mine && entry(i) < D ? __ldcg(src + entry(i)) : 0.f;
+    }
+  }
+  int which = 0;
+  for (int t0 = 0; t0 < q_len; t0 += TOKENS, which ^= 1) {
+    const int tokens = min(TOKENS, q_len - t0);
+    const bool more = t0 + TOKENS < q_len;
+    if (more) stage(t0 + TOKENS, which ^ 1);
+    if (more) copy_async_wait<1>(); else copy_async_wait<0>();
+    __syncthreads();
+    const float* k_rows = shared + which * buffer;
+    const float* q_rows = k_rows + TOKENS * pitch;
+    const float* v_rows = q_rows + TOKENS * pitch;
+    const float* coef = v_rows + TOKENS * COLS;
+    for (int t = 0; t < tokens; t += TB) {
+      float read[N];
+#pragma unroll
+      for (int n = 0; n < TB; ++n) {
+        const float2 gate = *reinterpret_cast<const float2*>(coef + (t + n) * COEF);      // keep, write
+        float u[C];
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          u[c] = gate.y * v_rows[(t + n) * COLS + group * C + c];
+          read[n * C + c] = 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < E; i += 4) {
+          const float4 k4 = *reinterpret_cast<const float4*>(k_rows + (t + n) * pitch + entry(i));
+          const float4 q4 = *reinterpret_cast<const float4*>(q_rows + (t + n) * pitch + entry(i));
+#pragma unroll
+          for (int c = 0; c < C; ++c) {
+            float sum = read[n * C + c];
+            S[c][i] = fmaf(k4.x, u[c], gate.x * S[c][i]);
+            sum = fmaf(q4.x, S[c][i], sum);
+            S[c][i + 1] = fmaf(k4.y, u[c], gate.x * S[c][i + 1]);
+            sum = fmaf(q4.y, S[c][i + 1], sum);
+            S[c][i + 2] = fmaf(k4.z, u[c], gate.x * S[c][i + 2]);
+            sum = fmaf(q4.z, S[c][i + 2], sum);
+            S[c][i + 3] = fmaf(k4.w, u[c], gate.x * S[c][i + 3]);
+            read[n * C + c] = fmaf(q4.w, S[c][i + 3], sum);
+          }
+        }
+      }
+      const int first = spread_sums<N, SL>(read, lane);
+      constexpr int HELD = N > SL ? N / SL : 1;
+      if (N >= SL || (s & (SL / N - 1)) == 0) {
+#pragma unroll
+        for (int i = 0; i < HELD; ++i) {
+          const int number = first + i, n = number / C, column = col0 + group * C + number % C;
+          if (t + n < tokens && column <= V) {
+            const size_t row_head = (size_t)(q_start + t0 + t + n) * p.heads + head;
+            if (column < V) p.reads[row_head * V + column] = read[i] * p.q_scale;
+            else p.norms[row_head] = read[i] * p.q_scale;
+          }
+        }
+      }
+    }
+    __syncthreads();      // the next turn of the loop stages into this buffer
+  }
+#pragma unroll
+  for (int c = 0; c < C; ++c) {
+    const int column = col0 + group * C + c;
+    if (column > V) continue;
+    float* dst = state + (size_t)column * D;
+    if (WIDE) {
+#pragma unroll
+      for (int i = 0; i < E; i += 4)
+        if (entry(i) < D) *reinterpret_cast<float4*>(dst + entry(i)) = make_float4(S[c][i], S[c][i + 1], S[c][i + 2], S[c][i + 3]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < E; ++i)
+        if (entry(i) < D) dst[entry(i)] = S[c][i];
+    }
+  }
+}
+
+template <int E, int SL, int C, bool WIDE, int THREADS = 128>
+static int launch_scan(const MemoryArgs& p, int segments, cudaStream_t stream) {
+  constexpr int COLS = THREADS / SL * C, TOKENS = SL == 32 ? 16 : 32;
+  constexpr size_t shared = sizeof(float) * 2 * (size_t)TOKENS * (2 * E * SL + COLS + 4);
+  static_assert(shared <= 227 * 1024, "staging buffers");
+  auto kernel = matrix_memory_scan_kernel<E, SL, C, WIDE, THREADS>;
+  if (shared > 48 * 1024) {
+    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+    if (err != cudaSuccess) return (int)err;
+  }
+  launch_kernel(kernel, dim3(segments, p.heads, (p.vdim + 1 + COLS - 1) / COLS), dim3(THREADS), shared, stream, p);
+  return launch_status();
+}
+
+// ------------------------------------------------------------------ normaliser, head norm, weight, gate
+// A warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(128)
+matrix_memory_finish_kernel(MemoryArgs p, T* __restrict__ out, long long items) {
+  pdl_trigger();
+  pdl_wait();
+  const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (item >= items) return;
+  const int lane = threadIdx.x & 31, V = p.vdim;
+  const long long row = item / p.heads;
+  const int head = (int)(item - row * p.heads);
+  const float* reads = p.reads + item * V;
+  const float* gate = p.gate + row * p.gate_stride + (size_t)head * V;
+  const float* weight = p.weight + (size_t)head * V;
+  const float inverse = 1.f / (fmaxf(fabsf(__ldcg(p.norms + item)), __ldcg(&p.coef[item].z)) + p.guard);
+  constexpr int HELD = 8;      // channels a lane keeps in registers
+  float o[HELD], g[HELD], sq = 0.f;
+#pragma unroll
+  for (int j = 0; j < HELD; ++j) {
+    const int c = lane + 32 * j;
+    o[j] = c < V ? __ldcg(reads + c) * inverse : 0.f;
+    g[j] = c < V ? __ldcg(gate + c) : 0.f;
+    sq = fmaf(o[j], o[j], sq);
+  }
+  for (int c = lane + 32 * HELD; c < V; c += 32) {
+    const float x = __ldcg(reads + c) * inverse;
+    sq = fmaf(x, x, sq);
+  }
+  const float factor = 1.f / sqrtf(warp_sum(sq) / (float)V + p.eps);
+  T* dst = out + item * V;
+#pragma unroll
+  for (int j = 0; j < HELD; ++j) {
+    const int c = lane + 32 * j;
+    if (c < V) dst[c] = from_float<T>(o[j] * factor * weight[c] * sigmoid(g[j]));
+  }
+  for (int c = lane + 32 * HELD; c < V; c += 32)
+    dst[c] = from_float<T>(__ldcg(reads + c) * inverse * factor * weight[c] * sigmoid(__ldcg(gate + c)));
+}
+
+template <typename T>
+static int launch_memory(const MemoryArgs& p, T* out, int rows, int segments, int max_q_len, bool wide, cudaStream_t stream) {
+  const int D = p.dim;
+  if (max_q_len == 1) {
+    const dim3 grid(segments, p.heads);
+    const size_t shared = sizeof(float) * (size_t)(p.vdim + 1);
+    if (!wide) launch_kernel(matrix_memory_decode_kernel<T, 0>, grid, dim3(DECODE_THREADS), shared, stream, p, out);
+    else if (D <= 128) launch_kernel(matrix_memory_decode_kernel<T, 1>, grid, dim3(DECODE_THREADS), shared, stream, p, out);
+    else if (D <= 256) launch_kernel(matrix_memory_decode_kernel<T, 2>, grid, dim3(DECODE_THREADS), shared, stream, p, out);
+    else launch_kernel(matrix_memory_decode_kernel<T, 4>, grid, dim3(DECODE_THREADS), shared, stream, p, out);
+    return launch_status();
+  }
+  if (p.coef == nullptr || p.reads == nullptr || p.norms == nullptr) return MLR_BAD_SIZE;
+  launch_kernel(matrix_memory_gates_kernel, dim3(segments, p.heads), dim3(GATE_THREADS), 0, stream, p);
+  int status = launch_status();
+  if (status != MLR_OK) return status;
+  if (wide) {
+    if (D <= 32) status = launch_scan<4, 8, 1, true>(p, segments, stream);
+    else if (D <= 64) status = launch_scan<4, 16, 1, true>(p, segments, stream);
+    else if (D <= 128) status = launch_scan<8, 16, 2, true>(p, segments, stream);
+    else if (D <= 256) status = launch_scan<8, 32, 2, true>(p, segments, stream);
+    else status = launch_scan<16, 32, 2, true>(p, segments, stream);
+  } else {
+    if (D <= 32) status = launch_scan<4, 8, 1, false>(p, segments, stream);
+    else if (D <= 128) status = launch_scan<16, 8, 1, false>(p, segments, stream);
+    else status = launch_scan<16, 32, 1, false>(p, segments, stream);
+  }
+  if (status != MLR_OK) return status;
+  const long long items = (long long)rows * p.heads;
+  launch_kernel(matrix_memory_finish_kernel<T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, p, out, items);
+  return launch_status();
+}
+
+}  // namespace mlr
+
+using namespace mlr;
+
+MLR_DEFINE_PDL_SWITCH
+
+// q, k: float32 rows of heads * dim entries; v, gate: rows of heads * vdim; i_raw, f_raw: rows of `heads` entries (each
+// with its own row stride); i_bias, f_bias: float32 [heads]; weight: float32 [heads * vdim]; coef: float32 scratch
+// [rows, heads, 4], reads: [rows, heads, vdim], norms: [rows, heads] (all three null for steps of single rows); states:
+// float32 [slots, heads, vdim + 1, dim], maxima: float32 [slots, heads]; out: [rows, heads * vdim] in `dtype`.
+// max_q_len: the longest segment of the step.
+MLR_EXPORT int mlr_matrix_memory(const float* q, long long q_stride, const float* k, long long k_stride, const float* v,
+                                 long long v_stride, const float* i_raw, long long i_stride, const float* f_raw,
+                                 long long f_stride, const float* gate, long long gate_stride, const float* i_bias,
+                                 const float* f_bias, const float* weight, float* coef, float* reads, float* norms,
+                                 float* states, float* maxima, void* out, const int* seg_q_start, const int* seg_q_len,
+                                 const int* seg_slot, int rows, int segments, int max_q_len, int heads, int dim, int vdim,
+                                 float cap, float guard, float eps, float q_scale, int dtype, cudaStream_t stream) {
+  if (segments == 0 || rows == 0) return MLR_OK;
+  if (segments < 0 || rows < 0 || max_q_len <= 0 || heads <= 0 || dim <= 0 || vdim <= 0 || !(cap > 0.f)) return MLR_BAD_SIZE;
+  if (dim > 512 || vdim > 4096 || heads > 65535 || segments > 65535) return MLR_TOO_LARGE;
+  MemoryArgs p{q, k, v, i_raw, f_raw, gate, q_stride, k_stride, v_stride, i_stride, f_stride, gate_stride, i_bias, f_bias,
+               weight, reinterpret_cast<float4*>(coef), reads, norms, states, maxima, seg_q_start, seg_q_len, seg_slot, heads,
+               dim, vdim, cap, guard, eps, q_scale};
+  auto multiple = [](long long n) { return n % 4 == 0; };
+  auto aligned = [](const void* ptr) { return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0; };
+  if (!aligned(coef)) return MLR_BAD_ALIGNMENT;
+  const bool wide = multiple(dim) && multiple(vdim) && multiple(q_stride) && multiple(k_stride) && multiple(v_stride) &&
+                    aligned(q) && aligned(k) && aligned(v) && aligned(states);
+  if (dtype == MLR_F32) return launch_memory(p, (float*)out, rows, segments, max_q_len, wide, stream);
+  if (dtype == MLR_BF16) return launch_memory(p, (bf16*)out, rows, segments, max_q_len, wide, stream);
+  return MLR_BAD_DTYPE;
+}

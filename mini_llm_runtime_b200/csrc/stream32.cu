@@ -20,6 +20,7 @@
 // mlr_clamped_gate         y = g * sigmoid(slope * g) * (u + 1) with g = min(gate, limit) and
 //                          u = clamp(up, -limit, limit), on rows of gate/up blocks.
 // mlr_scale_inplace        x *= s for float32 x (logit scale).
+// mlr_softcap_inplace      x <- cap tanh(x / cap) for float32 x (logit cap).
 #include "common.cuh"
 
 #include <type_traits>
@@ -505,6 +506,13 @@ __global__ void __launch_bounds__(256) scale_inplace_kernel(float* x, long long 
   if (index < count) x[index] *= factor;
 }
 
+__global__ void __launch_bounds__(256) softcap_inplace_kernel(float* x, long long count, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  const long long index = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (index < count) x[index] = cap * tanhf(x[index] / cap);
+}
+
 }  // namespace mlr
 
 using namespace mlr;
@@ -673,6 +681,15 @@ MLR_EXPORT int mlr_clamped_gate(const void* x, void* out, long long rows, int in
                   rows, inner, block, limit, slope);
   else
     return MLR_BAD_DTYPE;
+  return launch_status();
+}
+
+MLR_EXPORT int mlr_softcap_inplace(float* x, long long count, float cap, cudaStream_t stream) {
+  if (count == 0) return MLR_OK;
+  if (count < 0 || !(cap > 0.f)) return MLR_BAD_SIZE;
+  const long long blocks = (count + 255) / 256;
+  if (blocks > 0x7fffffffLL) return MLR_TOO_LARGE;
+  launch_kernel(softcap_inplace_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, count, cap);
   return launch_status();
 }
 

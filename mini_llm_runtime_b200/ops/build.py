@@ -55,6 +55,7 @@ LIBRARIES: dict[str, tuple[str, ...]] = {
     "state_space": (),
     "delta_rule": (),
     "attention_shaped_mma": (),
+    "matrix_memory": (),
 }
 
 _loaded: dict[str, ctypes.CDLL] = {}

@@ -1069,20 +1069,26 @@ class CudaOps:
             ctypes.c_float(slope), _code(gate_up.dtype), _stream()), "clamped_gate")
         return out
 
-    def linear_clamped_gate(self, x: torch.Tensor, weight: torch.Tensor, block: int, limit: float, slope: float) -> torch.Tensor:
-        """The clamped gate of (x Wg^T, x Wu^T) for ``weight`` [2*inner, K] of interleaved gate/up blocks."""
+    def linear_clamped_gate(self, x: torch.Tensor, weight: torch.Tensor, block: int, limit: float, slope: float,
+                            bias: torch.Tensor | None = None) -> torch.Tensor:
+        """The clamped gate of (x Wg^T + bg, x Wu^T + bu) for ``weight`` [2*inner, K] (and ``bias`` [2*inner]) of
+        interleaved gate/up blocks."""
         _need(x, "x", dims=2)
         _need(weight, "weight", x.dtype, 2)
         if x.shape[1] != weight.shape[1] or weight.shape[0] % (2 * block):
             raise KernelError("linear_clamped_gate: shapes do not fit the interleaved gate/up layout")
+        if bias is not None:
+            _need(bias, "bias", x.dtype, 1)
+            if bias.shape[0] != weight.shape[0]:
+                raise KernelError("bias length differs from the weight's output rows")
         if (self.use_tensor_cores and self.use_fused_swiglu and block == self.SWIGLU_BLOCK and x.dtype == torch.bfloat16
                 and x.shape[1] % 8 == 0 and x.shape[0] > 0 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0
                 and not self._skinny_fits(x, weight)):
             # many rows: the gate in the tensor-core product's epilogue
-            out = self._linear_tcgen05(x, weight, None, torch.bfloat16, swiglu=3, gate=(float(limit), float(slope)))
+            out = self._linear_tcgen05(x, weight, bias, torch.bfloat16, swiglu=3, gate=(float(limit), float(slope)))
             if out is not None:
                 return out
-        return self.clamped_gate(self.linear(x, weight), block, limit, slope)
+        return self.clamped_gate(self.linear(x, weight, bias), block, limit, slope)
 
     def scale_(self, x: torch.Tensor, factor: float) -> torch.Tensor:
         """x *= factor in place (float32)."""
@@ -1091,17 +1097,26 @@ class CudaOps:
             _ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(factor), _stream()), "scale")
         return x
 
+    def softcap_(self, x: torch.Tensor, cap: float) -> torch.Tensor:
+        """x <- cap * tanh(x / cap) in place (float32)."""
+        _need(x, "x", torch.float32)
+        _check(build.load_library("stream32").mlr_softcap_inplace(
+            _ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(cap), _stream()), "softcap")
+        return x
+
     # ------------------------------------------------------------------ latent attention
     def latent_prepare(self, down: torch.Tensor, q_at: int, q_rank: int, c_at: int, rank: int, rot: int,
-                       q_weight: torch.Tensor, c_weight: torch.Tensor, eps: float, positions: torch.Tensor,
+                       q_weight: torch.Tensor | None, c_weight: torch.Tensor, eps: float, positions: torch.Tensor,
                        frequencies: torch.Tensor, interleaved: bool, slots: torch.Tensor, pool: torch.Tensor,
-                       write: bool = True) -> torch.Tensor:
+                       write: bool = True, magnitude: float = 1.0) -> torch.Tensor | None:
         """From the float32 product ``down`` [rows, n]: the RMS-normalised query latent (columns
-        q_at .. q_at + q_rank, returned in the pool's dtype), and into the cache at ``slots`` the
+        q_at .. q_at + q_rank, returned in the pool's dtype; None with q_rank 0), and into the cache at ``slots`` the
         RMS-normalised latent (columns c_at .. c_at + rank) followed by the next ``rot`` columns with
-        their first 2 * len(frequencies) entries turned by the rows' positions."""
+        their first 2 * len(frequencies) entries turned by the rows' positions (sine and cosine times
+        ``magnitude``)."""
         _need(down, "down", torch.float32, 2)
-        _need(q_weight, "q_weight", torch.float32, 1)
+        if q_rank:
+            _need(q_weight, "q_weight", torch.float32, 1)
         _need(c_weight, "c_weight", torch.float32, 1)
         _need(positions, "positions", torch.int32, 1)
         _need(frequencies, "frequencies", torch.float32, 1)
@@ -1109,20 +1124,21 @@ class CudaOps:
         _need(pool, "pool", None, 4)
         rows = down.shape[0]
         if (q_at < 0 or c_at < 0 or q_at + q_rank > down.shape[1] or c_at + rank + rot > down.shape[1]
-                or q_weight.shape[0] != q_rank or c_weight.shape[0] != rank):
+                or (q_rank and q_weight.shape[0] != q_rank) or c_weight.shape[0] != rank):
             raise KernelError("column ranges or norm weights do not fit the product")
         if pool.shape[1] != 1 or pool.shape[3] != rank + rot or slots.shape[0] != rows or positions.shape[0] != rows:
             raise KernelError(f"pool has shape {tuple(pool.shape)}, expected [pages, 1, page_size, {rank + rot}]; "
                               "one slot and one position per row")
-        q_latent = torch.empty((rows, q_rank), dtype=pool.dtype, device=down.device)
+        q_latent = torch.empty((rows, q_rank), dtype=pool.dtype, device=down.device) if q_rank else None
         _check(build.load_library("attention_latent").mlr_latent_prepare(
             _ptr(down), ctypes.c_longlong(down.stride(0)), q_at, q_rank, c_at, rank, rot, _ptr(q_weight), _ptr(c_weight),
             _ptr(positions), _ptr(frequencies), frequencies.shape[0], int(bool(interleaved)), _ptr(slots), _ptr(q_latent),
-            _ptr(pool), rows, ctypes.c_float(eps), int(bool(write)), _code(pool.dtype), _stream()), "latent_prepare")
+            _ptr(pool), rows, ctypes.c_float(eps), ctypes.c_float(magnitude), int(bool(write)), _code(pool.dtype),
+            _stream()), "latent_prepare")
         return q_latent
 
     def _head_linear(self, x, x_head, weight, heads, n, k, kn, out, out_head, mode=0, tail=0, positions=None,
-                     frequencies=None, interleaved=False, gate=None, gate_per_head=False):
+                     frequencies=None, interleaved=False, gate=None, gate_per_head=False, magnitude=1.0):
         rows = x.shape[0]
         if (not isinstance(x, torch.Tensor) or not x.is_cuda or x.dtype != torch.float32 or x.dim() != 2
                 or x.stride(1) != 1):
@@ -1143,20 +1159,22 @@ class CudaOps:
             _check(build.load_library("attention_latent_mma").mlr_head_linear_mma(
                 _ptr(x), ctypes.c_longlong(x.stride(0)), x_head, _ptr(weight), _ptr(out), ctypes.c_longlong(out.stride(0)),
                 out_head, rows, heads, n, k, int(kn), mode, tail, pairs, int(bool(interleaved)), _ptr(positions),
-                _ptr(frequencies), gate_ptr, gate_row, int(bool(gate_per_head)), _code(out.dtype), _stream()),
+                _ptr(frequencies), ctypes.c_float(magnitude), gate_ptr, gate_row, int(bool(gate_per_head)), _code(out.dtype),
+                _stream()),
                 "head_linear (tensor cores)")
             return out
         _check(build.load_library("attention_latent").mlr_head_linear(
             _ptr(x), ctypes.c_longlong(x.stride(0)), x_head, _ptr(weight), _ptr(out), ctypes.c_longlong(out.stride(0)),
             out_head, rows, heads, n, k, int(kn), mode, tail, pairs, int(bool(interleaved)), _ptr(positions),
-            _ptr(frequencies), gate_ptr, gate_row, int(bool(gate_per_head)), _code(weight.dtype), _code(out.dtype),
-            _stream()), "head_linear")
+            _ptr(frequencies), ctypes.c_float(magnitude), gate_ptr, gate_row, int(bool(gate_per_head)), _code(weight.dtype),
+            _code(out.dtype), _stream()), "head_linear")
         return out
 
     def absorb_queries(self, q: torch.Tensor, weight: torch.Tensor, heads: int, dim: int, rot: int, rank: int,
-                       positions: torch.Tensor, frequencies: torch.Tensor, interleaved: bool) -> torch.Tensor:
-        """Queries into the latent space.  q: float32 [rows, heads * (dim + rot)], per head [plain | to be
-        turned]; weight [heads * dim, rank] (the per-head key matrix).  Returns, in the weight's dtype,
+                       positions: torch.Tensor, frequencies: torch.Tensor, interleaved: bool,
+                       magnitude: float = 1.0) -> torch.Tensor:
+        """Queries into the latent space.  q: float32 view [rows, heads * (dim + rot)], per head [plain | to be
+        turned] (sine and cosine times ``magnitude``); weight [heads * dim, rank] (the per-head key matrix).  Returns, in the weight's dtype,
         [rows, heads * (rank + rot)]: per head weight_h^T q_plain followed by the turned part."""
         _need(positions, "positions", torch.int32, 1)
         _need(frequencies, "frequencies", torch.float32, 1)
@@ -1164,18 +1182,18 @@ class CudaOps:
             raise KernelError("q does not match the head count and sizes")
         out = torch.empty((q.shape[0], heads * (rank + rot)), dtype=weight.dtype, device=q.device)
         return self._head_linear(q, dim + rot, weight, heads, rank, dim, True, out, rank + rot, mode=1, tail=rot,
-                                 positions=positions, frequencies=frequencies, interleaved=interleaved)
+                                 positions=positions, frequencies=frequencies, interleaved=interleaved, magnitude=magnitude)
 
     def latent_values(self, mixed: torch.Tensor, weight: torch.Tensor, heads: int, vdim: int, rank: int,
-                      gate: torch.Tensor, gate_per_head: bool) -> torch.Tensor:
+                      gate: torch.Tensor | None, gate_per_head: bool) -> torch.Tensor:
         """Per head weight_h [vdim, rank] applied to the attention's latent sums (mixed: float32
         [rows, heads * rank]), times sigmoid(gate) (float32 [rows, heads * vdim], or [rows, heads]
-        with ``gate_per_head``).  Returns [rows, heads * vdim] in the weight's dtype."""
+        with ``gate_per_head``; None: no gate).  Returns [rows, heads * vdim] in the weight's dtype."""
         if mixed.shape[1] != heads * rank:
             raise KernelError("mixed does not match the head count and latent size")
         out = torch.empty((mixed.shape[0], heads * vdim), dtype=weight.dtype, device=mixed.device)
-        return self._head_linear(mixed, rank, weight, heads, vdim, rank, False, out, vdim, mode=2, gate=gate,
-                                 gate_per_head=gate_per_head)
+        return self._head_linear(mixed, rank, weight, heads, vdim, rank, False, out, vdim, mode=0 if gate is None else 2,
+                                 gate=gate, gate_per_head=gate_per_head)
 
     use_latent_decode_kernel = True
     latent_decode_chunk_tiles = 4      # key tiles (of 32 keys) a CTA of the decode attention takes at least
@@ -1577,8 +1595,8 @@ class CudaOps:
     # ------------------------------------------------------------------ softmax attention with shaped scores
     SHAPED_CHUNK_TILES = 4      # key tiles (of 32 keys) a CTA of the tensor-core decode kernel takes at least
 
-    def shaped_attention(self, q: torch.Tensor, key: torch.Tensor, value: torch.Tensor | None, slots: torch.Tensor,
-                         k_pool: torch.Tensor, v_pool: torch.Tensor, batch: AttentionBatch, heads: int, kv_heads: int,
+    def shaped_attention(self, q: torch.Tensor, key: torch.Tensor | None, value: torch.Tensor | None, slots: torch.Tensor,
+                         k_pool: torch.Tensor, v_pool: torch.Tensor | None, batch: AttentionBatch, heads: int, kv_heads: int,
                          dim: int, vdim: int, scale: float, *, softcap: float = 0.0, slopes: torch.Tensor | None = None,
                          window: int = 0, chunk: int = 0, sink: torch.Tensor | None = None,
                          gate: torch.Tensor | None = None, write_kv: bool = True) -> torch.Tensor:
@@ -1586,9 +1604,10 @@ class CudaOps:
         score x = softcap * tanh(q . k * scale / softcap) (q . k * scale without a cap) - slopes_h * (i - j); position
         i sees the keys j <= i of its own chunk of ``chunk`` positions (0: no chunks) and of its last ``window``
         positions (0: all); exp(sink_h) joins each head's denominator; the result is multiplied by
-        sigmoid(gate).  q [rows, heads*dim], key [rows, kv_heads*dim], value [rows, kv_heads*vdim] or None (the
-        keys are the values: nothing else is cached), gate [rows, heads*vdim] or None: views with unit column
-        stride in the pools' dtype; slopes, sink: float32 [heads]."""
+        sigmoid(gate).  ``v_pool`` None: the keys are the values, nothing else is cached.  q [rows, heads*dim], key
+        [rows, kv_heads*dim] and value [rows, kv_heads*vdim] (both only with ``write_kv``; without it they are in
+        the pools already), gate [rows, heads*vdim] or None: views with unit column stride in the pools' dtype;
+        slopes, sink: float32 [heads]."""
         rows = q.shape[0]
         _need(k_pool, "k_pool", None, 4)
         dtype = k_pool.dtype
@@ -1605,7 +1624,9 @@ class CudaOps:
                     raise KernelError(f"{name}: one number per head")
         if slots.shape[0] != rows or k_pool.shape[1] != kv_heads or k_pool.shape[3] != dim:
             raise KernelError("one slot per row; the key pool must match the head count and size")
-        shared = value is None
+        shared = v_pool is None
+        if write_kv and (key is None or (value is None) != shared):
+            raise KernelError("nothing to store: keys, and values unless the keys are the values")
         if shared:
             if vdim != dim:
                 raise KernelError("keys that are values have one size")
@@ -1618,13 +1639,13 @@ class CudaOps:
             raise KernelError("the batch carries no attention work lists (plan_attention)")
         out = torch.empty((rows, heads * vdim), dtype=dtype, device=q.device)
         page_size = k_pool.shape[2]
-        on_tensor_cores = (shared and self.use_mma_attention and dtype == torch.bfloat16
+        on_tensor_cores = (vdim == dim and self.use_mma_attention and dtype == torch.bfloat16
                            and self._shaped_mma_fits(dim)
-                           and all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in (q, key))
+                           and all(t is None or (t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0) for t in (q, key))
                            and (gate is None or (gate.data_ptr() % 4 == 0 and gate.stride(0) % 2 == 0))
                            and batch.num_decode * heads <= self.ATTENTION_COUNTERS)
         only_decode = batch.num_decode == batch.num_segments
-        fused_store = on_tensor_cores and only_decode and write_kv      # the decode kernel stores the new keys itself
+        fused_store = on_tensor_cores and shared and only_decode and write_kv      # the decode kernel stores the new keys itself
         if write_kv and not fused_store:
             for rows_in, pool, size in ((key, k_pool, dim), (value, v_pool, vdim)):
                 if rows_in is not None:
@@ -1648,7 +1669,7 @@ class CudaOps:
         def launch(decode, fresh, lists, count, partial, counters, splits, what):
             _check(lib.mlr_attention_shaped_mma(
                 int(decode), *q_view, _ptr(fresh), ctypes.c_longlong(0 if fresh is None else fresh.stride(0)), _ptr(slots),
-                _ptr(k_pool), _ptr(out), *gate_view, _ptr(slopes), _ptr(sink), *lists, count, *segments, heads, kv_heads, dim,
+                _ptr(k_pool), _ptr(None if shared else v_pool), _ptr(out), *gate_view, _ptr(slopes), _ptr(sink), *lists, count, *segments, heads, kv_heads, dim,
                 page_size, int(window), int(chunk), ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(partial),
                 _ptr(counters), splits, _stream()), what)
 
@@ -1673,7 +1694,7 @@ class CudaOps:
                 # no item of 128 rows sees more keys than its rows' reach
                 longest = min(longest, min(int(chunk) or 1 << 30, int(window) or 1 << 30) + 128)
             _check(build.load_library("attention_tcgen05").mlr_attention_shaped_prefill_tcgen05(
-                *q_view, _ptr(k_pool), _ptr(out), _ptr(batch.plan["big_tile_seg"]), _ptr(batch.plan["big_tile_row0"]),
+                *q_view, _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(batch.plan["big_tile_seg"]), _ptr(batch.plan["big_tile_row0"]),
                 *segments, batch.counts["big"], rows, heads, kv_heads, dim, page_size, k_pool.shape[0], int(window), int(chunk),
                 ctypes.c_float(scale), ctypes.c_float(softcap), _ptr(slopes), _ptr(sink), *gate_view, longest,
                 _ptr(space["prefill_queue"]), _ptr(space["error_word"]),
@@ -1690,6 +1711,83 @@ class CudaOps:
         if dim not in cache:
             cache[dim] = bool(build.load_library("attention_shaped_mma").mlr_attention_shaped_mma_fits(dim))
         return cache[dim]
+
+    def head_prepare(self, q: torch.Tensor, key: torch.Tensor, value: torch.Tensor, positions: torch.Tensor,
+                     q_weight: torch.Tensor | None, k_weight: torch.Tensor | None, eps: float, freq: torch.Tensor | None,
+                     magnitude: float, interleaved: bool, slots: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
+                     heads: int, kv_heads: int, dim: int, vdim: int, write_kv: bool = True) -> torch.Tensor:
+        """Divide every q and k head by its root mean square over ``dim`` times a weight [dim] (None for both: not),
+        turn their first 2 * len(freq) entries by the rows' positions (sine and cosine times ``magnitude``; pairs
+        (2i, 2i + 1) with ``interleaved``, else half the turned entries apart), store k and the values as they are at
+        ``slots`` of the pools and return q [rows, heads*dim].  q [rows, heads*dim], key [rows, kv_heads*dim], value
+        [rows, kv_heads*vdim]: views with unit column stride in the pools' dtype."""
+        rows = q.shape[0]
+        _need(k_pool, "k_pool", None, 4)
+        _need(v_pool, "v_pool", k_pool.dtype, 4)
+        for name, view, width in (("q", q, heads * dim), ("key", key, kv_heads * dim), ("value", value, kv_heads * vdim)):
+            if not view.is_cuda or view.dtype != k_pool.dtype or tuple(view.shape) != (rows, width) or view.stride(1) != 1:
+                raise KernelError(f"{name} must be a CUDA view [{rows}, {width}] of {k_pool.dtype} with unit column stride")
+        _need(positions, "positions", torch.int32, 1)
+        _need(slots, "slots", torch.int64, 1)
+        if (q_weight is None) != (k_weight is None):
+            raise KernelError("norms on queries and keys, or on neither")
+        for name, vector in (("q_weight", q_weight), ("k_weight", k_weight)):
+            if vector is not None:
+                _need(vector, name, torch.float32, 1)
+                if vector.shape[0] != dim:
+                    raise KernelError(f"{name} holds {vector.shape[0]} entries, heads have {dim}")
+        if freq is not None:
+            _need(freq, "freq", torch.float32, 1)
+        rot = 0 if freq is None else 2 * freq.shape[0]
+        if rot > dim or positions.shape[0] != rows or slots.shape[0] != rows:
+            raise KernelError("at most dim turned entries; one position and one slot per row")
+        if (k_pool.shape[1] != kv_heads or k_pool.shape[3] != dim or v_pool.shape[:3] != k_pool.shape[:3]
+                or v_pool.shape[3] != vdim):
+            raise KernelError("page pools do not match the head sizes")
+        out = torch.empty((rows, heads * dim), dtype=k_pool.dtype, device=q.device)
+        views = [part for view in (q, key, value) for part in (_ptr(view), ctypes.c_longlong(view.stride(0)))]
+        _check(build.load_library("attention_rotated").mlr_head_prepare(
+            *views, _ptr(positions), _ptr(q_weight), _ptr(k_weight), _ptr(freq), _ptr(slots), _ptr(out), _ptr(k_pool),
+            _ptr(v_pool), rows, heads, kv_heads, dim, vdim, rot, int(bool(interleaved)), ctypes.c_float(eps),
+            ctypes.c_float(magnitude), k_pool.shape[2], int(bool(write_kv)), _code(k_pool.dtype), _stream()), "head_prepare")
+        return out
+
+    # ------------------------------------------------------------------ matrix memory
+    def matrix_memory(self, q, k, v, i_raw, f_raw, i_bias, f_bias, cap: float, guard: float, gate, weight: torch.Tensor,
+                      eps: float, state: torch.Tensor, maximum: torch.Tensor, ctx, heads: int, dim: int, vdim: int,
+                      out_dtype: torch.dtype) -> torch.Tensor:
+        """Per request and head, token after token, with i = cap tanh((i_raw + i_bias) / cap) and f = logsigmoid(cap
+        tanh((f_raw + f_bias) / cap)): m_t = max(f + m_{t-1}, i), S_t = e^(f + m_{t-1} - m_t) S_{t-1} + e^(i - m_t) k v^T, n_t
+        likewise with k alone, o = S_t^T q' / (max(|n_t . q'|, e^(-m_t)) + guard), q' = q * dim^-0.5; returns o / rms(o) *
+        weight * sigmoid(gate) [rows, heads*vdim] in ``out_dtype`` (rms over a head's entries, eps inside the root).
+        q, k [rows, heads*dim], v, gate [rows, heads*vdim], i_raw, f_raw [rows, heads]: float32 views with unit column
+        stride; weight float32 [heads*vdim]; state float32 [slots, heads, vdim + 1, dim] (the transposed S, n behind
+        it) and maximum float32 [slots, heads] are advanced in place."""
+        rows = q.shape[0]
+        for name, vector, size in (("i_bias", i_bias, heads), ("f_bias", f_bias, heads), ("weight", weight, heads * vdim)):
+            _need(vector, name, torch.float32, 1)
+            if vector.shape[0] != size:
+                raise KernelError(f"{name} holds {vector.shape[0]} entries, expected {size}")
+        _need(state, "state", torch.float32, 4)
+        _need(maximum, "maximum", torch.float32, 2)
+        if tuple(state.shape[1:]) != (heads, vdim + 1, dim) or tuple(maximum.shape) != (state.shape[0], heads):
+            raise KernelError(f"state has shape {tuple(state.shape)}, expected [slots, {heads}, {vdim + 1}, {dim}] and "
+                              "one maximum per slot and head")
+        out = torch.empty((rows, heads * vdim), dtype=out_dtype, device=q.device)
+        coef = reads = norms = None
+        if ctx.max_q_len > 1:
+            coef = torch.empty((rows, heads, 4), dtype=torch.float32, device=q.device)
+            reads = torch.empty((rows, heads * vdim), dtype=torch.float32, device=q.device)
+            norms = torch.empty((rows, heads), dtype=torch.float32, device=q.device)
+        _check(build.load_library("matrix_memory").mlr_matrix_memory(
+            *self._view(q, "q", rows, heads * dim), *self._view(k, "k", rows, heads * dim),
+            *self._view(v, "v", rows, heads * vdim), *self._view(i_raw, "i_raw", rows, heads),
+            *self._view(f_raw, "f_raw", rows, heads), *self._view(gate, "gate", rows, heads * vdim), _ptr(i_bias),
+            _ptr(f_bias), _ptr(weight), _ptr(coef), _ptr(reads), _ptr(norms), _ptr(state), _ptr(maximum), _ptr(out),
+            _ptr(ctx.seg_q_start), _ptr(ctx.seg_q_len), _ptr(ctx.seg_slot), rows, ctx.num_segments, int(ctx.max_q_len), heads,
+            dim, vdim, ctypes.c_float(cap), ctypes.c_float(guard), ctypes.c_float(eps), ctypes.c_float(float(dim) ** -0.5),
+            _code(out_dtype), _stream()), "matrix_memory")
+        return out
 
     # ------------------------------------------------------------------ gated delta rule
     def delta_rule_scan(self, q, k, v, a, b, dt_bias, A_log, state, ctx, heads: int, kv_heads: int, dim: int, vdim: int,

@@ -167,7 +167,7 @@ def test_shaped_attention_kernels_against_their_formula(heads, kv_heads, dim, sh
             k.use_mma_attention = use_mma
             try:
                 got = k.shaped_attention(xd[:, :heads * dim], xd[:, heads * dim:(heads + kv_heads) * dim], None, slots.to(DEVICE), pool,
-                                         pool, batch, heads, kv_heads, dim, dim, scale, softcap=softcap, window=window, chunk=chunk,
+                                         None, batch, heads, kv_heads, dim, dim, scale, softcap=softcap, window=window, chunk=chunk,
                                          gate=gate, **on_device)
             finally:
                 k.use_mma_attention = True
