@@ -76,7 +76,7 @@ def parse_args():
     parser.add_argument("--gemm", default=None, metavar="M,N,K[,swiglu]",
                         help="time this engine's bfloat16 product x[M,K] W[N,K]^T on one shape (weights rotate over "
                              "copies larger than L2) and print a small JSON record; nothing else runs")
-    parser.add_argument("--arch", choices=("qwen2", "zazasun", "rozesun", "bopilorn", "ratilorn", "vetevik"), default="qwen2",
+    parser.add_argument("--arch", choices=("qwen2", "zazasun", "rozesun", "bopilorn", "ratilorn", "vetevik", "zugarax"), default="qwen2",
                         help="zazasun: prefill and decode of the Zazasun architecture at a few layer sizes beside "
                              "Qwen2 at equal sizes, and its kernels alone against their rooflines (one JSON line "
                              "of its own; the default workload is untouched)")
@@ -772,6 +772,9 @@ def main():
     if args.arch == "vetevik":
         import bench_vetevik
         return bench_vetevik.run(args, sys.modules[__name__])
+    if args.arch == "zugarax":
+        import bench_zugarax
+        return bench_zugarax.run(args, sys.modules[__name__])
     return run_ours(args)
 
 
