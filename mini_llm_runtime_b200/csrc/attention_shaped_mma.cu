@@ -138,46 +138,6 @@ __device__ __forceinline__ void shaped_softmax_step(float (*s)[4], float (*o)[4]
   }
 }
 
-// S[16 x 8 NT] = Q K^T over a key tile whose rows are D + 8 apart (an odd number of 16-byte pieces: ldmatrix is
-// free of bank conflicts).
-template <int D, int NT>
-__device__ __forceinline__ void padded_qk(float (*s)[4], const uint32_t (*q_frag)[4], const bf16* tile, int lane) {
-#pragma unroll
-  for (int j = 0; j < NT; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
-#pragma unroll
-  for (int ks = 0; ks < D / 16; ++ks) {
-#pragma unroll
-    for (int jp = 0; jp < NT / 2; ++jp) {
-      uint32_t b[4];
-      const int key = jp * 16 + (lane & 7) + ((lane >> 4) << 3);
-      ldmatrix_x4(b, tile + key * (D + 8) + (ks * 2 + ((lane >> 3) & 1)) * 8);
-      mma_bf16(s[2 * jp], q_frag[ks], b[0], b[1]);
-      mma_bf16(s[2 * jp + 1], q_frag[ks], b[2], b[3]);
-    }
-  }
-}
-
-// O[16 x D] += P V with V the same tile.
-template <int D, int NT>
-__device__ __forceinline__ void padded_pv(float (*o)[4], const float (*p)[4], const bf16* tile, int lane) {
-#pragma unroll
-  for (int kk = 0; kk < NT / 2; ++kk) {
-    uint32_t a[4];
-    a[0] = pack_bf16(p[2 * kk][0], p[2 * kk][1]);
-    a[1] = pack_bf16(p[2 * kk][2], p[2 * kk][3]);
-    a[2] = pack_bf16(p[2 * kk + 1][0], p[2 * kk + 1][1]);
-    a[3] = pack_bf16(p[2 * kk + 1][2], p[2 * kk + 1][3]);
-#pragma unroll
-    for (int dp = 0; dp < D / 16; ++dp) {
-      uint32_t b[4];
-      const int key = kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
-      ldmatrix_x4_trans(b, tile + key * (D + 8) + (dp * 2 + (lane >> 4)) * 8);
-      mma_bf16(o[2 * dp], a, b[0], b[1]);
-      mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
-    }
-  }
-}
-
 // Row of the pool (in units of D entries) that holds a key of one kv head, or -1.
 __device__ __forceinline__ int pool_row(const ShapedArgs& p, const int* table, int key, int kv_head) {
   const int logical = p.page_shift >= 0 ? key >> p.page_shift : key / p.page_size;

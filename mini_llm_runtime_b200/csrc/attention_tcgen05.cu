@@ -156,6 +156,7 @@ __device__ __forceinline__ void fa_wait(uint64_t* bar, uint32_t parity, int* err
 struct FaScore {
   float in_scale, out_scale;        // capped: scale / cap and cap * log2(e); else scale * log2(e) and 1
   int capped, chunk;                // chunk 0: none
+  int bent;                         // scores need more than a positive factor, which the softmax itself applies
   const float *slopes, *sinks;      // [heads] or null
   const bf16* gate;                 // rows of heads * D, or null
   long long gate_stride;
@@ -222,9 +223,13 @@ __device__ __forceinline__ void fa_shape_scores(float (&s)[FA_KEYS], const FaSco
 __device__ __forceinline__ void fa_gate32(float* v, const bf16* gate) {
 #pragma unroll
   for (int c = 0; c < 32; c += 8) {
-    uint4 raw;      // gate rows start at even columns only: four loads of two
-    const unsigned int* src = reinterpret_cast<const unsigned int*>(gate + c);
-    raw.x = __ldcg(src); raw.y = __ldcg(src + 1); raw.z = __ldcg(src + 2); raw.w = __ldcg(src + 3);
+    uint4 raw;
+    if ((reinterpret_cast<uintptr_t>(gate) & 15) == 0) {
+      raw = __ldcg(reinterpret_cast<const uint4*>(gate + c));
+    } else {      // gate rows are sure to start at even columns only: four loads of two
+      const unsigned int* src = reinterpret_cast<const unsigned int*>(gate + c);
+      raw.x = __ldcg(src); raw.y = __ldcg(src + 1); raw.z = __ldcg(src + 2); raw.w = __ldcg(src + 3);
+    }
     const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -467,6 +472,11 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
       const int warp_first = first_pos + warp * 32;
       const int warp_lo = lowest_of(first_pos + min(rows - 1, warp * 32 + 31));
       const float slope2 = SHAPED && score.slopes != nullptr ? score.slopes[head] * 1.4426950408889634f : 0.f;
+      if (SHAPED && score.gate != nullptr && r < rows) {      // on its way to the L2 while the keys are walked
+        const bf16* gate = score.gate + (size_t)(q_start + row0 + r) * score.gate_stride + (size_t)head * D;
+#pragma unroll
+        for (int c = 0; c < D; c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(gate + c));
+      }
       float m_run = -INFINITY;      // the running max of the scaled scores (base-2 exponent)
       float m_base = -INFINITY;     // the exponent that sum, probabilities and output are relative to
       float l = 0.f;
@@ -484,7 +494,7 @@ prefill_attention_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
         fa_tmem_wait_ld();
         fa_fence_before();
 
-        if (SHAPED) fa_shape_scores(s, score, slope2, slope2 * (float)(key0 - position));
+        if (SHAPED && score.bent) fa_shape_scores(s, score, slope2, slope2 * (float)(key0 - position));
         if (!(warp_full && key0 + FA_KEYS - 1 <= warp_first && key0 >= warp_lo)) {
 #pragma unroll
           for (int c = 0; c < FA_KEYS; ++c) {
@@ -750,7 +760,7 @@ static int fa_launch(const void* q, const void* k_pool, const void* v_pool, void
   const int ctas = (int)(units < resident ? units : resident);
   launch_kernel(prefill_attention_tcgen05_kernel<D, SHAPED>, dim3(ctas), dim3(FA_THREADS), shared, stream, q_map, k_map, v_map,
                 (bf16*)out, tile_seg, tile_row0, seg_q_start, seg_q_len, seg_pos0, block_table, seg_slot, table_width, tiles, heads,
-                kv_heads, page_size, page_shift, window, SHAPED ? 1.f : scale * 1.4426950408889634f, queue, error_word, max_parts,
+                kv_heads, page_size, page_shift, window, SHAPED && score.bent ? 1.f : scale * 1.4426950408889634f, queue, error_word, max_parts,
                 tiles_per_unit, (float*)scratch, counters, (int)shared, score);
   return launch_status();
 }
@@ -819,6 +829,7 @@ MLR_EXPORT int mlr_attention_shaped_prefill_tcgen05(
   const float log2e = 1.4426950408889634f;
   FaScore score;
   score.capped = softcap > 0.f;
+  score.bent = score.capped || slopes != nullptr || !(scale > 0.f);
   score.in_scale = score.capped ? scale / softcap : scale * log2e;
   score.out_scale = score.capped ? softcap * log2e : 1.f;
   score.chunk = chunk;

@@ -15,7 +15,19 @@
 //                               own rounding does to S cancels out.
 // matrix_memory_scan_kernel     the recurrence of longer segments, token after token, value channels over blocks.
 // matrix_memory_finish_kernel   normaliser, head norm, weight and gate of the scan's rows.
-#include "common.cuh"
+//
+// In bfloat16, prompts take chunks of 64 tokens through the tensor cores instead of the token-by-token scan.  q, k and
+// v are projections and enter rounded to bfloat16; everything else stays 32-bit: products of a 32-bit operand are
+// taken of its three bfloat16 parts (24 bits), sums are 32-bit.  With K_t the product of the keeps of a chunk's tokens up to
+// t and D_ts = write_s times the keeps of s + 1 .. t (products of numbers up to one, no differences of logarithms),
+//
+//   S^T q_t (of token t) = K_t S_before^T q_t + sum_{s <= t} A_ts v_s    with  A_ts = D_ts (k_s . q_t)
+//   S_behind = K_last S_before + sum_s k_s (D_last,s v_s)^T
+//
+// matrix_memory_pairs_kernel    all chunks at once: A, D_last and K of every chunk, q, k and v as bfloat16.
+// matrix_memory_chunks_kernel   the chunks of a (request, head) one after the other, value channels over blocks; the
+//                               state stays in registers as accumulators.
+#include "mma_attention.cuh"
 #include "copy_async.cuh"
 #include "lane_sums.cuh"
 
@@ -29,6 +41,9 @@ struct MemoryArgs {
   float4* coef;                         // [rows, heads]: keep, write, e^(-m), unused
   float* reads;                         // [rows, heads, vdim]: S^T q before the normaliser
   float* norms;                         // [rows, heads]: n . q
+  float* pairs;                         // chunks: [rows, heads, 64], A
+  float2* factors;                      // chunks: [rows, heads]: D_last and K
+  bf16 *q16, *k16, *v16;                // chunks: [rows, heads * dim], the same, [rows, heads * vdim]
   float* states;                        // [slots, heads, vdim + 1, dim]
   float* maxima;                        // [slots, heads]
   const int *seg_q_start, *seg_q_len, *seg_slot;
@@ -402,6 +417,314 @@ static int launch_scan(const MemoryArgs& p, int segments, cudaStream_t stream) {
   return launch_status();
 }
 
+// ------------------------------------------------------------------ chunks on the tensor cores
+constexpr int CHUNK = 64;         // tokens
+constexpr int CHUNK_COLS = 32;    // value channels of a block of the sequential kernel
+constexpr int CHUNK_PITCH = CHUNK_COLS + 8;
+
+__device__ __forceinline__ uint2 pack4(float4 x) { return make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w)); }
+
+// grid: (chunks, heads, segments)
+template <int D>
+__global__ void __launch_bounds__(128)
+matrix_memory_pairs_kernel(MemoryArgs p) {
+  constexpr int PITCH = D + 8;
+  extern __shared__ __align__(16) uint8_t raw[];
+  bf16* q_tile = reinterpret_cast<bf16*>(raw);               // [64][PITCH]
+  bf16* k_tile = q_tile + CHUNK * PITCH;
+  float (*decay)[CHUNK + 1] = reinterpret_cast<float (*)[CHUNK + 1]>(k_tile + CHUNK * PITCH);
+  __shared__ float keep[CHUNK], write[CHUNK];
+  const int head = blockIdx.y, seg = blockIdx.z, V = p.vdim;
+  const int t0 = blockIdx.x * CHUNK, count = min(CHUNK, p.seg_q_len[seg] - t0);
+  if (count <= 0) return;
+  const size_t row0 = (size_t)p.seg_q_start[seg] + t0;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  pdl_wait();
+  if (threadIdx.x < CHUNK) {      // a place without a token keeps everything and writes nothing
+    float2 gate = make_float2(1.f, 0.f);
+    if (threadIdx.x < count) gate = __ldcg(reinterpret_cast<const float2*>(p.coef + (row0 + threadIdx.x) * p.heads + head));
+    keep[threadIdx.x] = gate.x;
+    write[threadIdx.x] = gate.y;
+  }
+  for (int idx = threadIdx.x; idx < CHUNK * (D / 4); idx += 128) {
+    const int r = idx / (D / 4), d = (idx - r * (D / 4)) << 2;
+    uint2 q2 = make_uint2(0u, 0u), k2 = q2;
+    if (r < count) {
+      const size_t at = (row0 + r) * p.heads * D + (size_t)head * D + d;
+      q2 = pack4(__ldcg(reinterpret_cast<const float4*>(p.q + (row0 + r) * p.q_stride + (size_t)head * D + d)));
+      k2 = pack4(__ldcg(reinterpret_cast<const float4*>(p.k + (row0 + r) * p.k_stride + (size_t)head * D + d)));
+      *reinterpret_cast<uint2*>(p.q16 + at) = q2;
+      *reinterpret_cast<uint2*>(p.k16 + at) = k2;
+    }
+    *reinterpret_cast<uint2*>(q_tile + r * PITCH + d) = q2;
+    *reinterpret_cast<uint2*>(k_tile + r * PITCH + d) = k2;
+  }
+  for (int idx = threadIdx.x; idx < count * (V / 4); idx += 128) {
+    const int r = idx / (V / 4), c = (idx - r * (V / 4)) << 2;
+    *reinterpret_cast<uint2*>(p.v16 + (row0 + r) * p.heads * V + (size_t)head * V + c) =
+        pack4(__ldcg(reinterpret_cast<const float4*>(p.v + (row0 + r) * p.v_stride + (size_t)head * V + c)));
+  }
+  __syncthreads();
+  // a thread per column of D: its writing token's share at every later token
+  if (threadIdx.x < CHUNK) {
+    const int s = threadIdx.x;
+    float x = write[s];
+    for (int t = 0; t < CHUNK; ++t) {
+      if (t > s) x *= keep[t];
+      decay[t][s] = t >= s ? x : 0.f;
+    }
+    if (s < count) p.factors[(row0 + s) * p.heads + head].x = x;      // places behind the last token keep it
+  } else if (threadIdx.x == CHUNK) {
+    float x = 1.f;
+    for (int t = 0; t < count; ++t) {
+      x *= keep[t];
+      p.factors[(row0 + t) * p.heads + head].y = x;
+    }
+  }
+  uint32_t q_frag[D / 16][4];
+#pragma unroll
+  for (int ks = 0; ks < D / 16; ++ks)
+    ldmatrix_x4(q_frag[ks], q_tile + (warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * PITCH + (ks * 2 + (lane >> 4)) * 8);
+  float s[CHUNK / 8][4];
+  padded_qk<D, CHUNK / 8>(s, q_frag, k_tile, lane);
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int t = warp * 16 + (lane >> 2) + 8 * i;
+    if (t >= count) continue;
+    float* dst = p.pairs + ((row0 + t) * p.heads + head) * CHUNK;
+#pragma unroll
+    for (int j = 0; j < CHUNK / 8; ++j) {
+      const int c = j * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(dst + c) = make_float2(s[j][2 * i] * decay[t][c], s[j][2 * i + 1] * decay[t][c + 1]);
+    }
+  }
+}
+
+// the three bfloat16 parts of a pair of numbers
+__device__ __forceinline__ void split_pair(float x, float y, uint32_t* part) {
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {
+    const __nv_bfloat162 rounded = __floats2bfloat162_rn(x, y);
+    part[i] = *reinterpret_cast<const uint32_t*>(&rounded);
+    const float2 back = __bfloat1622float2(rounded);
+    x -= back.x;
+    y -= back.y;
+  }
+}
+
+// c[0 .. 3] (four blocks of 8 columns) += a * tile, tile: 16 rows from `row` of a [..][CHUNK_PITCH] tile
+__device__ __forceinline__ void mma_cols(float (*c)[4], const uint32_t* a, const bf16* tile, int row, int lane) {
+#pragma unroll
+  for (int dp = 0; dp < CHUNK_COLS / 16; ++dp) {
+    uint32_t b[4];
+    ldmatrix_x4_trans(b, tile + (row + (lane & 7) + (((lane >> 3) & 1) << 3)) * CHUNK_PITCH + (dp * 2 + (lane >> 4)) * 8);
+    mma_bf16(c[2 * dp], a, b[0], b[1]);
+    mma_bf16(c[2 * dp + 1], a, b[2], b[3]);
+  }
+}
+
+// grid: (segments, heads, blocks of 32 state rows).  Warp w keeps the key channels w D / 4 .. of the state.
+template <int D>
+__global__ void __launch_bounds__(128)
+matrix_memory_chunks_kernel(MemoryArgs p) {
+  pdl_trigger();
+  constexpr int PITCH = D + 8, MT = D / 64, NT = CHUNK_COLS / 8, PIECES = D / 8;
+  extern __shared__ __align__(16) uint8_t raw[];
+  bf16* qk_tiles = reinterpret_cast<bf16*>(raw);                       // 2 x (queries, keys) [64][PITCH]
+  bf16* v_tiles = qk_tiles + 4 * CHUNK * PITCH;                         // 2 x [64][CHUNK_PITCH]
+  bf16* s_parts = v_tiles + 2 * CHUNK * CHUNK_PITCH;                    // 3 x [D][CHUNK_PITCH]
+  bf16* w_parts = s_parts + 3 * D * CHUNK_PITCH;                        // 3 x [64][CHUNK_PITCH]
+  float2* factors = reinterpret_cast<float2*>(w_parts + 3 * CHUNK * CHUNK_PITCH);      // 2 x [64]
+  const int seg = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * CHUNK_COLS, V = p.vdim;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int q_start = p.seg_q_start[seg], q_len = p.seg_q_len[seg];
+  float* state = p.states + ((size_t)p.seg_slot[seg] * p.heads + head) * (size_t)(V + 1) * D;
+  // value channels beyond the last: the normaliser's is one, the others zero; no copy overwrites them
+  for (int idx = threadIdx.x; idx < 2 * CHUNK * CHUNK_COLS; idx += 128) {
+    const int r = idx / CHUNK_COLS, c = idx - r * CHUNK_COLS;
+    if (col0 + c >= V) v_tiles[r * CHUNK_PITCH + c] = __float2bfloat16_rn(col0 + c == V ? 1.f : 0.f);
+  }
+  pdl_wait();
+  auto stage = [&](int t0, int which) {
+    const int count = min(CHUNK, q_len - t0);
+    const size_t row0 = (size_t)q_start + t0;
+    bf16* q_tile = qk_tiles + which * 2 * CHUNK * PITCH;
+    bf16* k_tile = q_tile + CHUNK * PITCH;
+    for (int idx = threadIdx.x; idx < CHUNK * PIECES; idx += 128) {
+      const int r = idx / PIECES, c = (idx - r * PIECES) * 8;
+      const bool valid = r < count;
+      const size_t at = valid ? (row0 + r) * p.heads * D + (size_t)head * D + c : 0;
+      cp_async_16(q_tile + r * PITCH + c, p.q16 + at, valid);
+      cp_async_16(k_tile + r * PITCH + c, p.k16 + at, valid);
+    }
+    for (int idx = threadIdx.x; idx < CHUNK * (CHUNK_COLS / 8); idx += 128) {
+      const int r = idx / (CHUNK_COLS / 8), c = (idx - r * (CHUNK_COLS / 8)) * 8;
+      if (col0 + c >= V) continue;
+      const bool valid = r < count;
+      cp_async_16(v_tiles + (which * CHUNK + r) * CHUNK_PITCH + c,
+                  p.v16 + (valid ? (row0 + r) * p.heads * V + (size_t)head * V + col0 + c : 0), valid);
+    }
+    cp_async_commit();
+    if (threadIdx.x < CHUNK)      // a place without a token writes nothing
+      factors[which * CHUNK + threadIdx.x] =
+          threadIdx.x < count ? __ldcg(p.factors + (row0 + threadIdx.x) * p.heads + head) : make_float2(0.f, 0.f);
+  };
+  stage(0, 0);
+  float S[MT][NT][4];      // accumulators: key channel (row) lane / 4 + 8 (e / 2), value channel (column) 2 (lane % 4) + e % 2
+  auto place = [&](int mt, int nt, int e, int* d, int* c) {
+    *d = warp * (D / 4) + mt * 16 + (lane >> 2) + 8 * (e >> 1);
+    *c = col0 + nt * 8 + (lane & 3) * 2 + (e & 1);
+  };
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        int d, c;
+        place(mt, nt, e, &d, &c);
+        S[mt][nt][e] = c <= V ? __ldcg(state + (size_t)c * D + d) : 0.f;
+      }
+  int which = 0;
+  for (int t0 = 0; t0 < q_len; t0 += CHUNK, which ^= 1) {
+    const int count = min(CHUNK, q_len - t0);
+    const size_t row0 = (size_t)q_start + t0;
+    cp_async_wait<0>();
+    __syncthreads();      // this chunk is here, and everybody is done with the one before
+    if (t0 + CHUNK < q_len) stage(t0 + CHUNK, which ^ 1);
+    const bf16* q_tile = qk_tiles + which * 2 * CHUNK * PITCH;
+    const bf16* k_tile = q_tile + CHUNK * PITCH;
+    const bf16* v_tile = v_tiles + which * CHUNK * CHUNK_PITCH;
+    const float2* factor = factors + which * CHUNK;
+    // this warp's rows of A, asked for early: keys up to the rows' own chunk part only
+    const int r0 = warp * 16 + (lane >> 2);
+    const float* a_row[2] = {p.pairs + ((row0 + r0) * p.heads + head) * CHUNK + (lane & 3) * 2,
+                             p.pairs + ((row0 + r0 + 8) * p.heads + head) * CHUNK + (lane & 3) * 2};
+    float2 a_pair[CHUNK / 16][4];
+#pragma unroll
+    for (int ks = 0; ks < CHUNK / 16; ++ks)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        a_pair[ks][e] = make_float2(0.f, 0.f);
+        if (ks <= warp && r0 + 8 * (e & 1) < count)
+          a_pair[ks][e] = __ldcg(reinterpret_cast<const float2*>(a_row[e & 1] + ks * 16 + 8 * (e >> 1)));
+      }
+    // the state and the weighed values in parts
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          uint32_t part[3];
+          split_pair(S[mt][nt][2 * i], S[mt][nt][2 * i + 1], part);
+          int d, c;
+          place(mt, nt, 2 * i, &d, &c);
+#pragma unroll
+          for (int n = 0; n < 3; ++n)
+            *reinterpret_cast<uint32_t*>(s_parts + (n * D + d) * CHUNK_PITCH + (c - col0)) = part[n];
+        }
+    for (int idx = threadIdx.x; idx < CHUNK * (CHUNK_COLS / 2); idx += 128) {
+      const int r = idx / (CHUNK_COLS / 2), c = (idx - r * (CHUNK_COLS / 2)) * 2;
+      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v_tile + r * CHUNK_PITCH + c));
+      const float weight = factor[r].x;
+      uint32_t part[3];
+      split_pair(weight * v.x, weight * v.y, part);
+#pragma unroll
+      for (int n = 0; n < 3; ++n) *reinterpret_cast<uint32_t*>(w_parts + (n * CHUNK + r) * CHUNK_PITCH + c) = part[n];
+    }
+    __syncthreads();
+    // reads: of the state before the chunk, then of the chunk's own tokens
+    float o[NT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
+    if (warp * 16 < count) {
+#pragma unroll
+      for (int ks = 0; ks < D / 16; ++ks) {
+        uint32_t a[4];
+        ldmatrix_x4(a, q_tile + (warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * PITCH + (ks * 2 + (lane >> 4)) * 8);
+#pragma unroll
+        for (int n = 2; n >= 0; --n) mma_cols(o, a, s_parts + n * D * CHUNK_PITCH, ks * 16, lane);      // smallest part first
+      }
+      const float before[2] = {factor[r0].y, factor[r0 + 8].y};
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[nt][e] *= before[e >> 1];
+#pragma unroll
+      for (int ks = 0; ks < CHUNK / 16; ++ks) {
+        if (ks > warp) continue;
+        uint32_t part[4][3];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split_pair(a_pair[ks][e].x, a_pair[ks][e].y, part[e]);
+#pragma unroll
+        for (int n = 2; n >= 0; --n) {
+          const uint32_t a[4] = {part[0][n], part[1][n], part[2][n], part[3][n]};
+          mma_cols(o, a, v_tile, ks * 16, lane);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        if (r0 + 8 * i >= count) continue;
+        const size_t row_head = (row0 + r0 + 8 * i) * p.heads + head;
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          const int c = col0 + nt * 8 + (lane & 3) * 2;
+          if (c < V)
+            *reinterpret_cast<float2*>(p.reads + row_head * V + c) = make_float2(o[nt][2 * i] * p.q_scale, o[nt][2 * i + 1] * p.q_scale);
+          else if (c == V)
+            p.norms[row_head] = o[nt][2 * i] * p.q_scale;
+        }
+      }
+    }
+    // the state behind the chunk
+    const float kept = factor[count - 1].y;
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[mt][nt][e] *= kept;
+#pragma unroll
+      for (int ks = 0; ks < CHUNK / 16; ++ks) {
+        uint32_t a[4];      // keys transposed: channels are the product's rows
+        ldmatrix_x4_trans(a, k_tile + (ks * 16 + ((lane >> 4) << 3) + (lane & 7)) * PITCH + warp * (D / 4) + mt * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int n = 2; n >= 0; --n) mma_cols(S[mt], a, w_parts + n * CHUNK * CHUNK_PITCH, ks * 16, lane);
+      }
+    }
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        int d, c;
+        place(mt, nt, e, &d, &c);
+        if (c <= V) state[(size_t)c * D + d] = S[mt][nt][e];
+      }
+}
+
+template <int D>
+static int launch_chunks(const MemoryArgs& p, int segments, int max_q_len, cudaStream_t stream) {
+  constexpr size_t shared = sizeof(bf16) * (size_t)(4 * CHUNK * (D + 8) + (2 * CHUNK + 3 * D + 3 * CHUNK) * CHUNK_PITCH) +
+                            sizeof(float2) * 2 * CHUNK;
+  static_assert(shared <= 227 * 1024, "tiles");
+  constexpr size_t pairs_shared = sizeof(bf16) * (size_t)(2 * CHUNK * (D + 8)) + sizeof(float) * CHUNK * (CHUNK + 1);
+  cudaError_t err = cudaFuncSetAttribute(matrix_memory_chunks_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);
+  if (err == cudaSuccess)
+    err = cudaFuncSetAttribute(matrix_memory_pairs_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)pairs_shared);
+  if (err != cudaSuccess) return (int)err;
+  launch_kernel(matrix_memory_pairs_kernel<D>, dim3((max_q_len + CHUNK - 1) / CHUNK, p.heads, segments), dim3(128), pairs_shared,
+                stream, p);
+  const int status = launch_status();
+  if (status != MLR_OK) return status;
+  launch_kernel(matrix_memory_chunks_kernel<D>, dim3(segments, p.heads, (p.vdim + CHUNK_COLS) / CHUNK_COLS), dim3(128), shared, stream, p);
+  return launch_status();
+}
+
 // ------------------------------------------------------------------ normaliser, head norm, weight, gate
 // A warp per (row, head).
 template <typename T>
@@ -442,6 +765,8 @@ matrix_memory_finish_kernel(MemoryArgs p, T* __restrict__ out, long long items) 
     dst[c] = from_float<T>(__ldcg(reads + c) * inverse * factor * weight[c] * sigmoid(__ldcg(gate + c)));
 }
 
+static bool chunks_fit(int dim, int vdim) { return (dim == 64 || dim == 128) && vdim % 8 == 0; }
+
 template <typename T>
 static int launch_memory(const MemoryArgs& p, T* out, int rows, int segments, int max_q_len, bool wide, cudaStream_t stream) {
   const int D = p.dim;
@@ -458,7 +783,10 @@ static int launch_memory(const MemoryArgs& p, T* out, int rows, int segments, in
   launch_kernel(matrix_memory_gates_kernel, dim3(segments, p.heads), dim3(GATE_THREADS), 0, stream, p);
   int status = launch_status();
   if (status != MLR_OK) return status;
-  if (wide) {
+  if (p.pairs != nullptr) {
+    if (!wide || !chunks_fit(D, p.vdim)) return MLR_BAD_SIZE;
+    status = D == 64 ? launch_chunks<64>(p, segments, max_q_len, stream) : launch_chunks<128>(p, segments, max_q_len, stream);
+  } else if (wide) {
     if (D <= 32) status = launch_scan<4, 8, 1, true>(p, segments, stream);
     else if (D <= 64) status = launch_scan<4, 16, 1, true>(p, segments, stream);
     else if (D <= 128) status = launch_scan<8, 16, 2, true>(p, segments, stream);
@@ -481,27 +809,37 @@ using namespace mlr;
 
 MLR_DEFINE_PDL_SWITCH
 
+// Whether prompts of these head sizes can go through the tensor cores in chunks (with `pairs`).
+MLR_EXPORT int mlr_matrix_memory_chunks_fit(int dim, int vdim) { return chunks_fit(dim, vdim); }
+
 // q, k: float32 rows of heads * dim entries; v, gate: rows of heads * vdim; i_raw, f_raw: rows of `heads` entries (each
 // with its own row stride); i_bias, f_bias: float32 [heads]; weight: float32 [heads * vdim]; coef: float32 scratch
-// [rows, heads, 4], reads: [rows, heads, vdim], norms: [rows, heads] (all three null for steps of single rows); states:
+// [rows, heads, 4], reads: [rows, heads, vdim], norms: [rows, heads] (all three null for steps of single rows); pairs:
+// float32 scratch [rows, heads, 64 + 2] and packed: bfloat16 scratch [rows, heads, 2 dim + vdim] (both or neither: chunks
+// on the tensor cores, or the token-by-token scan; 16-byte aligned); states:
 // float32 [slots, heads, vdim + 1, dim], maxima: float32 [slots, heads]; out: [rows, heads * vdim] in `dtype`.
 // max_q_len: the longest segment of the step.
 MLR_EXPORT int mlr_matrix_memory(const float* q, long long q_stride, const float* k, long long k_stride, const float* v,
                                  long long v_stride, const float* i_raw, long long i_stride, const float* f_raw,
                                  long long f_stride, const float* gate, long long gate_stride, const float* i_bias,
                                  const float* f_bias, const float* weight, float* coef, float* reads, float* norms,
-                                 float* states, float* maxima, void* out, const int* seg_q_start, const int* seg_q_len,
+                                 float* pairs, void* packed, float* states, float* maxima, void* out, const int* seg_q_start, const int* seg_q_len,
                                  const int* seg_slot, int rows, int segments, int max_q_len, int heads, int dim, int vdim,
                                  float cap, float guard, float eps, float q_scale, int dtype, cudaStream_t stream) {
   if (segments == 0 || rows == 0) return MLR_OK;
   if (segments < 0 || rows < 0 || max_q_len <= 0 || heads <= 0 || dim <= 0 || vdim <= 0 || !(cap > 0.f)) return MLR_BAD_SIZE;
   if (dim > 512 || vdim > 4096 || heads > 65535 || segments > 65535) return MLR_TOO_LARGE;
+  bf16* q16 = (bf16*)packed;
+  bf16* k16 = q16 == nullptr ? nullptr : q16 + (size_t)rows * heads * dim;
+  bf16* v16 = q16 == nullptr ? nullptr : k16 + (size_t)rows * heads * dim;
+  if ((pairs == nullptr) != (packed == nullptr)) return MLR_BAD_SIZE;
   MemoryArgs p{q, k, v, i_raw, f_raw, gate, q_stride, k_stride, v_stride, i_stride, f_stride, gate_stride, i_bias, f_bias,
-               weight, reinterpret_cast<float4*>(coef), reads, norms, states, maxima, seg_q_start, seg_q_len, seg_slot, heads,
+               weight, reinterpret_cast<float4*>(coef), reads, norms, pairs,
+               pairs == nullptr ? nullptr : reinterpret_cast<float2*>(pairs + (size_t)rows * heads * CHUNK), q16, k16, v16, states, maxima, seg_q_start, seg_q_len, seg_slot, heads,
                dim, vdim, cap, guard, eps, q_scale};
   auto multiple = [](long long n) { return n % 4 == 0; };
   auto aligned = [](const void* ptr) { return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0; };
-  if (!aligned(coef)) return MLR_BAD_ALIGNMENT;
+  if (!aligned(coef) || !aligned(pairs) || !aligned(packed)) return MLR_BAD_ALIGNMENT;
   const bool wide = multiple(dim) && multiple(vdim) && multiple(q_stride) && multiple(k_stride) && multiple(v_stride) &&
                     aligned(q) && aligned(k) && aligned(v) && aligned(states);
   if (dtype == MLR_F32) return launch_memory(p, (float*)out, rows, segments, max_q_len, wide, stream);

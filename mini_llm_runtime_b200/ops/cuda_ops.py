@@ -1753,6 +1753,15 @@ class CudaOps:
         return out
 
     # ------------------------------------------------------------------ matrix memory
+    use_memory_chunks = True      # bfloat16 prompts in chunks of 64 tokens on the tensor cores
+    MEMORY_CHUNK_ROWS = 16        # longest portion of a step from which that pays
+
+    def _memory_chunks_fit(self, dim: int, vdim: int) -> bool:
+        cache = self.__dict__.setdefault("_memory_fits", {})
+        if (dim, vdim) not in cache:
+            cache[(dim, vdim)] = bool(build.load_library("matrix_memory").mlr_matrix_memory_chunks_fit(dim, vdim))
+        return cache[(dim, vdim)]
+
     def matrix_memory(self, q, k, v, i_raw, f_raw, i_bias, f_bias, cap: float, guard: float, gate, weight: torch.Tensor,
                       eps: float, state: torch.Tensor, maximum: torch.Tensor, ctx, heads: int, dim: int, vdim: int,
                       out_dtype: torch.dtype) -> torch.Tensor:
@@ -1774,8 +1783,13 @@ class CudaOps:
             raise KernelError(f"state has shape {tuple(state.shape)}, expected [slots, {heads}, {vdim + 1}, {dim}] and "
                               "one maximum per slot and head")
         out = torch.empty((rows, heads * vdim), dtype=out_dtype, device=q.device)
-        coef = reads = norms = None
+        coef = reads = norms = pairs = packed = None
         if ctx.max_q_len > 1:
+            if (out_dtype == torch.bfloat16 and self.use_memory_chunks and ctx.max_q_len >= self.MEMORY_CHUNK_ROWS
+                    and all(t.data_ptr() % 16 == 0 and t.stride(0) % 4 == 0 for t in (q, k, v))
+                    and self._memory_chunks_fit(dim, vdim)):
+                pairs = torch.empty((rows, heads, 66), dtype=torch.float32, device=q.device)
+                packed = torch.empty((rows, heads, 2 * dim + vdim), dtype=torch.bfloat16, device=q.device)
             coef = torch.empty((rows, heads, 4), dtype=torch.float32, device=q.device)
             reads = torch.empty((rows, heads * vdim), dtype=torch.float32, device=q.device)
             norms = torch.empty((rows, heads), dtype=torch.float32, device=q.device)
@@ -1783,7 +1797,8 @@ class CudaOps:
             *self._view(q, "q", rows, heads * dim), *self._view(k, "k", rows, heads * dim),
             *self._view(v, "v", rows, heads * vdim), *self._view(i_raw, "i_raw", rows, heads),
             *self._view(f_raw, "f_raw", rows, heads), *self._view(gate, "gate", rows, heads * vdim), _ptr(i_bias),
-            _ptr(f_bias), _ptr(weight), _ptr(coef), _ptr(reads), _ptr(norms), _ptr(state), _ptr(maximum), _ptr(out),
+            _ptr(f_bias), _ptr(weight), _ptr(coef), _ptr(reads), _ptr(norms), _ptr(pairs),
+            _ptr(packed), _ptr(state), _ptr(maximum), _ptr(out),
             _ptr(ctx.seg_q_start), _ptr(ctx.seg_q_len), _ptr(ctx.seg_slot), rows, ctx.num_segments, int(ctx.max_q_len), heads,
             dim, vdim, ctypes.c_float(cap), ctypes.c_float(guard), ctypes.c_float(eps), ctypes.c_float(float(dim) ** -0.5),
             _code(out_dtype), _stream()), "matrix_memory")

@@ -216,17 +216,18 @@ def test_windowed_attention_over_values_of_their_own(heads, kv_heads, dim, vdim,
 
 
 @pytest.mark.parametrize("heads,dim,vdim", [(4, 32, 24), (3, 64, 40), (4, 128, 36), (2, 200, 16), (2, 384, 12), (2, 10, 6), (3, 66, 33),
-                                            (2, 256, 20), (2, 128, 128), (1, 40, 300)])
+                                            (2, 256, 20), (2, 128, 128), (1, 40, 300), (3, 64, 64), (2, 128, 24), (5, 64, 40)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_matrix_memory_kernels_against_their_formula(heads, dim, vdim, dtype):
-    """A ragged batch whose requests go on over several steps with portions of every remainder of the kernel's block
-    of tokens, and steps of single rows; gates from shut to wide open, over long and short memories."""
+    """A ragged batch whose requests go on over several steps with portions of every remainder of the kernels' blocks
+    and chunks of tokens, and steps of single rows; gates from shut to wide open, over long and short memories; in
+    bfloat16 the sizes of 64 and 128 go through the tensor cores."""
     k = ops.current()
     generator = torch.Generator().manual_seed(dim + vdim)
     qk, inner, cap = heads * dim, heads * vdim, 9.0
     width = 2 * qk + 2 * inner + 2 * heads
     width += -width % 8
-    lengths = [[37, 1, 2, 300], [1, 3, 41, 5], [1, 1, 1, 1], [6, 70, 4, 1], [1, 1, 1, 1]]
+    lengths = [[37, 1, 2, 300], [1, 3, 41, 5], [1, 1, 1, 1], [6, 70, 4, 1], [1, 1, 1, 1], [64, 128, 65, 63]]
     total = [sum(col) for col in zip(*lengths)]
     sequences = [torch.randn(t, width, generator=generator) for t in total]
     at = 2 * qk + 2 * inner
