@@ -171,10 +171,10 @@ matrix_memory_decode_kernel(MemoryArgs p, T* __restrict__ out) {
 }
 
 // ------------------------------------------------------------------ gates of longer segments
-constexpr int GATE_THREADS = 256;
+constexpr int GATE_THREADS = 1024;
 constexpr int GATE_WARPS = GATE_THREADS / 32;
 
-// grid: (segments, heads).  256 tokens per turn.
+// grid: (segments, heads).  1,024 tokens per turn.
 __global__ void __launch_bounds__(GATE_THREADS)
 matrix_memory_gates_kernel(MemoryArgs p) {
   __shared__ float total_a[GATE_WARPS], total_b[GATE_WARPS], last[GATE_WARPS];
@@ -419,7 +419,7 @@ static int launch_scan(const MemoryArgs& p, int segments, cudaStream_t stream) {
 
 // ------------------------------------------------------------------ chunks on the tensor cores
 constexpr int CHUNK = 64;         // tokens
-constexpr int CHUNK_COLS = 32;    // value channels of a block of the sequential kernel
+constexpr int CHUNK_COLS = 16;    // value channels of a block of the sequential kernel
 constexpr int CHUNK_PITCH = CHUNK_COLS + 8;
 
 __device__ __forceinline__ uint2 pack4(float4 x) { return make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w)); }
@@ -565,10 +565,11 @@ matrix_memory_chunks_kernel(MemoryArgs p) {
       cp_async_16(v_tiles + (which * CHUNK + r) * CHUNK_PITCH + c,
                   p.v16 + (valid ? (row0 + r) * p.heads * V + (size_t)head * V + col0 + c : 0), valid);
     }
+    if (threadIdx.x < CHUNK) {      // a place without a token writes nothing
+      const bool valid = threadIdx.x < count;
+      copy_async_8(factors + which * CHUNK + threadIdx.x, p.factors + (valid ? (row0 + threadIdx.x) * p.heads + head : 0), valid);
+    }
     cp_async_commit();
-    if (threadIdx.x < CHUNK)      // a place without a token writes nothing
-      factors[which * CHUNK + threadIdx.x] =
-          threadIdx.x < count ? __ldcg(p.factors + (row0 + threadIdx.x) * p.heads + head) : make_float2(0.f, 0.f);
   };
   stage(0, 0);
   float S[MT][NT][4];      // accumulators: key channel (row) lane / 4 + 8 (e / 2), value channel (column) 2 (lane % 4) + e % 2
@@ -635,23 +636,27 @@ matrix_memory_chunks_kernel(MemoryArgs p) {
       for (int n = 0; n < 3; ++n) *reinterpret_cast<uint32_t*>(w_parts + (n * CHUNK + r) * CHUNK_PITCH + c) = part[n];
     }
     __syncthreads();
-    // reads: of the state before the chunk, then of the chunk's own tokens
-    float o[NT][4];
+    // reads: of the state before the chunk, then of the chunk's own tokens; a sum per part (short chains of products)
+    float o[3][NT][4];
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
+    for (int n = 0; n < 3; ++n)
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) o[n][nt][0] = o[n][nt][1] = o[n][nt][2] = o[n][nt][3] = 0.f;
     if (warp * 16 < count) {
 #pragma unroll
       for (int ks = 0; ks < D / 16; ++ks) {
         uint32_t a[4];
         ldmatrix_x4(a, q_tile + (warp * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * PITCH + (ks * 2 + (lane >> 4)) * 8);
 #pragma unroll
-        for (int n = 2; n >= 0; --n) mma_cols(o, a, s_parts + n * D * CHUNK_PITCH, ks * 16, lane);      // smallest part first
+        for (int n = 0; n < 3; ++n) mma_cols(o[n], a, s_parts + n * D * CHUNK_PITCH, ks * 16, lane);
       }
       const float before[2] = {factor[r0].y, factor[r0 + 8].y};
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt)
+      for (int n = 0; n < 3; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[nt][e] *= before[e >> 1];
+        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) o[n][nt][e] *= before[e >> 1];
 #pragma unroll
       for (int ks = 0; ks < CHUNK / 16; ++ks) {
         if (ks > warp) continue;
@@ -659,11 +664,15 @@ matrix_memory_chunks_kernel(MemoryArgs p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) split_pair(a_pair[ks][e].x, a_pair[ks][e].y, part[e]);
 #pragma unroll
-        for (int n = 2; n >= 0; --n) {
+        for (int n = 0; n < 3; ++n) {
           const uint32_t a[4] = {part[0][n], part[1][n], part[2][n], part[3][n]};
-          mma_cols(o, a, v_tile, ks * 16, lane);
+          mma_cols(o[n], a, v_tile, ks * 16, lane);
         }
       }
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[0][nt][e] += o[1][nt][e] + o[2][nt][e];
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         if (r0 + 8 * i >= count) continue;
@@ -672,9 +681,9 @@ matrix_memory_chunks_kernel(MemoryArgs p) {
         for (int nt = 0; nt < NT; ++nt) {
           const int c = col0 + nt * 8 + (lane & 3) * 2;
           if (c < V)
-            *reinterpret_cast<float2*>(p.reads + row_head * V + c) = make_float2(o[nt][2 * i] * p.q_scale, o[nt][2 * i + 1] * p.q_scale);
+            *reinterpret_cast<float2*>(p.reads + row_head * V + c) = make_float2(o[0][nt][2 * i] * p.q_scale, o[0][nt][2 * i + 1] * p.q_scale);
           else if (c == V)
-            p.norms[row_head] = o[nt][2 * i] * p.q_scale;
+            p.norms[row_head] = o[0][nt][2 * i] * p.q_scale;
         }
       }
     }
@@ -726,8 +735,11 @@ static int launch_chunks(const MemoryArgs& p, int segments, int max_q_len, cudaS
 }
 
 // ------------------------------------------------------------------ normaliser, head norm, weight, gate
-// A warp per (row, head).
-template <typename T>
+__device__ __forceinline__ void store4(float* dst, float4 y) { *reinterpret_cast<float4*>(dst) = y; }
+__device__ __forceinline__ void store4(bf16* dst, float4 y) { *reinterpret_cast<uint2*>(dst) = pack4(y); }
+
+// A warp per (row, head).  WIDE: at most 256 channels, in pieces of four (sizes, strides and pointers allow it).
+template <typename T, bool WIDE>
 __global__ void __launch_bounds__(128)
 matrix_memory_finish_kernel(MemoryArgs p, T* __restrict__ out, long long items) {
   pdl_trigger();
@@ -741,6 +753,31 @@ matrix_memory_finish_kernel(MemoryArgs p, T* __restrict__ out, long long items) 
   const float* gate = p.gate + row * p.gate_stride + (size_t)head * V;
   const float* weight = p.weight + (size_t)head * V;
   const float inverse = 1.f / (fmaxf(fabsf(__ldcg(p.norms + item)), __ldcg(&p.coef[item].z)) + p.guard);
+  if (WIDE) {
+    float4 o[2], g[2];
+    float sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int c = (lane + 32 * j) * 4;
+      o[j] = g[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < V) {
+        o[j] = __ldcg(reinterpret_cast<const float4*>(reads + c));
+        g[j] = __ldcg(reinterpret_cast<const float4*>(gate + c));
+      }
+      o[j].x *= inverse; o[j].y *= inverse; o[j].z *= inverse; o[j].w *= inverse;
+      sq += fmaf(o[j].x, o[j].x, o[j].y * o[j].y) + fmaf(o[j].z, o[j].z, o[j].w * o[j].w);
+    }
+    const float factor = 1.f / sqrtf(warp_sum(sq) / (float)V + p.eps);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int c = (lane + 32 * j) * 4;
+      if (c >= V) continue;
+      const float4 w = *reinterpret_cast<const float4*>(weight + c);
+      store4(out + item * V + c, make_float4(o[j].x * factor * w.x * sigmoid(g[j].x), o[j].y * factor * w.y * sigmoid(g[j].y),
+                                             o[j].z * factor * w.z * sigmoid(g[j].z), o[j].w * factor * w.w * sigmoid(g[j].w)));
+    }
+    return;
+  }
   constexpr int HELD = 8;      // channels a lane keeps in registers
   float o[HELD], g[HELD], sq = 0.f;
 #pragma unroll
@@ -799,7 +836,11 @@ static int launch_memory(const MemoryArgs& p, T* out, int rows, int segments, in
   }
   if (status != MLR_OK) return status;
   const long long items = (long long)rows * p.heads;
-  launch_kernel(matrix_memory_finish_kernel<T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, p, out, items);
+  auto aligned = [](const void* ptr) { return (reinterpret_cast<uintptr_t>(ptr) & 15) == 0; };
+  const bool pieces = p.vdim % 4 == 0 && p.vdim <= 256 && p.gate_stride % 4 == 0 && aligned(p.gate) && aligned(p.reads) &&
+                      aligned(p.weight) && aligned(out);
+  launch_kernel(pieces ? matrix_memory_finish_kernel<T, true> : matrix_memory_finish_kernel<T, false>,
+                dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, p, out, items);
   return launch_status();
 }
 
